@@ -99,7 +99,31 @@ __device__ __forceinline__ float apply_act(float v, int act) {
     if (act == 2) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));  // gelu (erf form)
     if (act == 3) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));  // gelu (tanh form)
     if (act == 4) return v / (1.f + expf(-v));                              // silu
+    if (act == 5) return v > 0.f ? v * v : 0.f;                             // the square of relu
     return v;
+}
+
+// Rotation by position of a pair (u, v): the pair turns by the angle a = pos * freq (float) and is multiplied by `amp`.
+struct Rotation {
+    const float* freq;      // one frequency per pair
+    int dims;               // the first `dims` dimensions of a vector turn, the others pass
+    int neighbours;         // 0: dimension i is paired with i + dims/2; 1: dimension 2i with 2i + 1
+    float amp;              // factor on sine and cosine
+};
+__device__ __forceinline__ int rot_partner(const Rotation& r, int e) {
+    const int half = r.dims >> 1;
+    return r.neighbours ? (e ^ 1) : (e < half ? e + half : e - half);
+}
+// dimension e (< dims) of the turned vector, from its own value x and its partner's y
+__device__ __forceinline__ float rot_apply(const Rotation& r, int e, int pos, float x, float y) {
+    const int half = r.dims >> 1;
+    const bool low = r.neighbours ? !(e & 1) : e < half;
+    const int i = r.neighbours ? (e >> 1) : (low ? e : e - half);
+    float sn, cs;
+    sincosf((float)pos * r.freq[i], &sn, &cs);
+    sn *= r.amp;
+    cs *= r.amp;
+    return low ? x * cs - y * sn : x * cs + y * sn;
 }
 
 static inline int st_launch_status() { return (int)cudaGetLastError(); }

@@ -8,7 +8,7 @@
 //   * a group takes the rows offsets[g]..offsets[g+1]-1 of a sorted list (the experts of a mixture): the launch walks
 //     row tiles (tile_group[i], tile_row0[i]) made on the device, arow = a_rows[row] / a_row_div where a_rows is
 //     given (the sorted (token, choice) items, a_row_div choices per token), else the row itself.
-// Epilogue: none, or "gated": w[g] holds 2 * n_out rows, gate rows first, and c = act(gate) * up.
+// Epilogue: c = act(product), or "gated": w[g] holds 2 * n_out rows, gate rows first, and c = act(gate) * up.
 //
 // gemm_grouped_mma: bfloat16 on the warp-level tensor cores (mma.sync m16n8k16, float accumulation): tiles of 64 rows
 // x 64 outputs x 64 of k, four warps of 32 x 32 each, rows gathered and weights streamed by 16-byte asynchronous
@@ -115,6 +115,8 @@ gemm_grouped_plain_kernel(const T* __restrict__ a, const T* __restrict__ w, TO* 
             if (sh.gated) {
                 // both products are rounded to the storage type first, as two separate products would leave them
                 v = apply_act(to_f32(from_f32<T>(v)), sh.act) * to_f32(from_f32<T>(acu[i][j]));
+            } else if (sh.act) {
+                v = apply_act(v, sh.act);
             }
             c[(long long)r * sh.ldc + g * sh.c_goff + n] = from_f32<TO>(v);
         }
@@ -261,6 +263,7 @@ gemm_grouped_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, 
                 if (r >= row_end || n >= sh.n_out) continue;
                 float v = acc[i][j][e];
                 if (GATED) v = apply_act(to_f32(from_f32<bf16>(v)), sh.act) * to_f32(from_f32<bf16>(acu[i][j][e]));
+                else if (sh.act) v = apply_act(v, sh.act);
                 c[(long long)r * sh.ldc + g * sh.c_goff + n] = from_f32<TO>(v);
             }
 }

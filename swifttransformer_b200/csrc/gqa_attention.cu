@@ -1,8 +1,8 @@
 // Grouped-query attention whose keys and values have sizes of their own, over the flat paged cache: the
 // preparation of queries, keys and values from a fused projection, and the plain attention kernel.
 //
-//   q, k   <- projection + bias; the first rot_dims dimensions of every head rotated by position, dimension i
-//             paired with i + rot_dims/2 (float angle p * inv_freq[i], sincosf); q times the temperature
+//   q, k   <- projection + bias; the first rot.dims dimensions of every head rotated by position (Rotation: halves or
+//             neighbours, float angle p * freq[i], sincosf); q times the temperature
 //             1 + coef * ln(floor((p + 1) / every) + 1)  (coef == 0: none)
 //   s_j    = scale * q . k_j over the keys the query sees (gqa_attention.cuh: a window of recent keys plus the
 //             first keep_first keys of the request, or all keys up to the query)
@@ -22,7 +22,7 @@
 template <typename T>
 __global__ void __launch_bounds__(GP_THREADS)
 gqa_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off, const float* __restrict__ bias,
-                   const float* __restrict__ inv_freq, int rot_dims, float temp_coef, int temp_every,
+                   Rotation rot, float temp_coef, int temp_every,
                    T* __restrict__ q_out, T* __restrict__ pool, DiffCache cache, const int* __restrict__ positions,
                    const int* __restrict__ seq_of_token, const int* __restrict__ slots,
                    const int* __restrict__ block_table, int nh, int write_kv, int* __restrict__ status) {
@@ -39,7 +39,6 @@ gqa_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int
         if (page < 0 && status && threadIdx.x == 0 && blockIdx.y == 0) *status = 1;
     }
     const int pip = pos % cache.page_size;
-    const int half = rot_dims / 2;
     const float temp = temp_coef != 0.f ? 1.f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.f) : 1.f;
     const T* row = proj + (size_t)t * ld;
     for (int c = blockIdx.y * GP_THREADS + threadIdx.x; c < qw + kw + vw; c += GP_THREADS * gridDim.y) {
@@ -55,13 +54,9 @@ gqa_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int
         const int head = cc / dim, e = cc % dim;
         const int col = (is_q ? q_off : k_off) + cc;
         float x = load1_cg(row + col) + (bias ? bias[col] : 0.f);
-        if (e < rot_dims) {
-            const bool low = e < half;
-            const int pcol = low ? col + half : col - half;
-            const float y = load1_cg(row + pcol) + (bias ? bias[pcol] : 0.f);
-            float sn, cs;
-            sincosf((float)pos * inv_freq[low ? e : e - half], &sn, &cs);
-            x = low ? x * cs - y * sn : x * cs + y * sn;
+        if (e < rot.dims) {
+            const int pcol = col - e + rot_partner(rot, e);
+            x = rot_apply(rot, e, pos, x, load1_cg(row + pcol) + (bias ? bias[pcol] : 0.f));
         }
         if (is_q) q_out[(size_t)t * qw + cc] = from_f32<T>(x * temp);
         else cache_keys(pool, cache, page, head, pip)[e] = from_f32<T>(x);
@@ -74,7 +69,7 @@ gqa_prepare_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int
 template <typename T>
 __global__ void __launch_bounds__(GP_THREADS)
 gqa_prepare_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off,
-                        const float* __restrict__ bias, const float* __restrict__ inv_freq, int rot_dims,
+                        const float* __restrict__ bias, Rotation rot,
                         float temp_coef, int temp_every, float norm_eps, T* __restrict__ q_out, T* __restrict__ pool,
                         DiffCache cache, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                         const int* __restrict__ slots, const int* __restrict__ block_table, int nh, int write_kv,
@@ -91,7 +86,6 @@ gqa_prepare_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
         if (page < 0 && status && threadIdx.x == 0 && blockIdx.y == 0) *status = 1;
     }
     const int pip = pos % cache.page_size;
-    const int half = rot_dims / 2;
     const float temp = temp_coef != 0.f ? 1.f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.f) : 1.f;
     const T* row = proj + (size_t)t * ld;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = GP_THREADS / 32;
@@ -118,13 +112,9 @@ gqa_prepare_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
             if (e >= dim) continue;
             const int col = col0 + e;
             float v = load1_cg(row + col) + (bias ? bias[col] : 0.f);
-            if (e < rot_dims) {
-                const bool low = e < half;
-                const int pcol = low ? col + half : col - half;
-                const float y = load1_cg(row + pcol) + (bias ? bias[pcol] : 0.f);
-                float sn, cs;
-                sincosf((float)pos * inv_freq[low ? e : e - half], &sn, &cs);
-                v = low ? v * cs - y * sn : v * cs + y * sn;
+            if (e < rot.dims) {
+                const int pcol = col - e + rot_partner(rot, e);
+                v = rot_apply(rot, e, pos, v, load1_cg(row + pcol) + (bias ? bias[pcol] : 0.f));
             }
             x[r] = v;
             ss = fmaf(v, v, ss);
@@ -145,12 +135,13 @@ ST_EXPORT int st_gqa_prepare(const void* proj, int ld, int q_off, int k_off, int
                              void* pool, long long page_stride, long long entry_offset, const int* positions,
                              const int* seq_of_token, const int* slots, const int* block_table, int max_pages,
                              int n_tokens, int nh, int nkv, int dim, int vd, int page_size, int write_kv, int* status,
-                             int dtype, void* stream, float norm_eps) {
+                             int dtype, void* stream, float norm_eps, int neighbours, float rot_amp) {
     if (n_tokens <= 0) return 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv || dim <= 0 || vd <= 0 || page_size <= 0) return ST_ERR_BAD_ARG;
     if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims > 0 && !inv_freq)) return ST_ERR_BAD_ARG;
     if (temp_coef != 0.f && temp_every <= 0) return ST_ERR_BAD_ARG;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
+    const Rotation rot = {inv_freq, rot_dims, neighbours, rot_amp};
     const int total = nh * dim + (write_kv ? nkv * (dim + vd) : 0);
     int gy = (total + GP_THREADS * 4 - 1) / (GP_THREADS * 4);
     if (gy > 64) gy = 64;
@@ -164,23 +155,23 @@ ST_EXPORT int st_gqa_prepare(const void* proj, int ld, int q_off, int k_off, int
         dim3 ngrid(n_tokens, ny);
         if (dtype == 0)
             return st_launch_pdl("gqa_prepare", gqa_prepare_norm_kernel<float>, ngrid, dim3(GP_THREADS), 0, s,
-                                 (const float*)proj, ld, q_off, k_off, v_off, bias, inv_freq, rot_dims, temp_coef,
+                                 (const float*)proj, ld, q_off, k_off, v_off, bias, rot, temp_coef,
                                  temp_every, norm_eps, (float*)q_out, (float*)pool, c, positions, seq_of_token, slots,
                                  block_table, nh, write_kv, status);
         if (dtype == 1)
             return st_launch_pdl("gqa_prepare", gqa_prepare_norm_kernel<bf16>, ngrid, dim3(GP_THREADS), 0, s,
-                                 (const bf16*)proj, ld, q_off, k_off, v_off, bias, inv_freq, rot_dims, temp_coef,
+                                 (const bf16*)proj, ld, q_off, k_off, v_off, bias, rot, temp_coef,
                                  temp_every, norm_eps, (bf16*)q_out, (bf16*)pool, c, positions, seq_of_token, slots,
                                  block_table, nh, write_kv, status);
         return ST_ERR_BAD_DTYPE;
     }
     if (dtype == 0)
         return st_launch_pdl("gqa_prepare", gqa_prepare_kernel<float>, grid, dim3(GP_THREADS), 0, s, (const float*)proj, ld,
-                             q_off, k_off, v_off, bias, inv_freq, rot_dims, temp_coef, temp_every, (float*)q_out,
+                             q_off, k_off, v_off, bias, rot, temp_coef, temp_every, (float*)q_out,
                              (float*)pool, c, positions, seq_of_token, slots, block_table, nh, write_kv, status);
     if (dtype == 1)
         return st_launch_pdl("gqa_prepare", gqa_prepare_kernel<bf16>, grid, dim3(GP_THREADS), 0, s, (const bf16*)proj, ld,
-                             q_off, k_off, v_off, bias, inv_freq, rot_dims, temp_coef, temp_every, (bf16*)q_out,
+                             q_off, k_off, v_off, bias, rot, temp_coef, temp_every, (bf16*)q_out,
                              (bf16*)pool, c, positions, seq_of_token, slots, block_table, nh, write_kv, status);
     return ST_ERR_BAD_DTYPE;
 }
@@ -274,7 +265,7 @@ gqa_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ pool, 
         const int e = threadIdx.x + c * GK;
         if (e >= vd) continue;
         float o = acc[c] * inv;
-        if (gate) o *= sigmoidf_(load1_cg(gate + (size_t)t * epi.gate_ld + h * vd + e));
+        if (gate) o *= sigmoidf_(load1_cg(gate + (size_t)t * epi.gate_ld + (epi.gate_heads ? h : h * vd + e)));
         out[((size_t)t * nh + h) * vd + e] = from_f32<T>(o);
     }
 }
@@ -284,13 +275,13 @@ ST_EXPORT int st_gqa_attention_plain(const void* q, const void* pool, long long 
                                      const int* slots, const int* block_table, int max_pages, int n_tokens, int nh,
                                      int nkv, int dim, int vd, int page_size, float scale, int window, int keep_first,
                                      int has_sink, float sink, const void* gate, long long gate_ld, float out_scale,
-                                     int* status, int dtype, void* stream, const float* sinks) {
+                                     int* status, int dtype, void* stream, const float* sinks, int gate_heads) {
     if (n_tokens <= 0) return 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv || dim <= 0 || vd <= 0 || page_size <= 0 || keep_first < 0) return ST_ERR_BAD_ARG;
     if (vd > G_VPASS * GK || dim > 4096) return ST_ERR_TOO_LARGE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
     const GqaMask mask = {window, keep_first};
-    const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr};
+    const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr, gate_heads};
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(n_tokens, nh);
     const size_t smem = (size_t)(dim + GK) * sizeof(float);
@@ -532,7 +523,7 @@ gqa_attention_single_kernel(const bf16* __restrict__ q, const bf16* __restrict__
             O *= c;
         }
         float o = L > 0.f ? O * epi.out_scale / L : 0.f;
-        if (gate) o *= sigmoidf_(load1_cg(gate + (size_t)t * epi.gate_ld + h * vd + e));
+        if (gate) o *= sigmoidf_(load1_cg(gate + (size_t)t * epi.gate_ld + (epi.gate_heads ? h : h * vd + e)));
         out[((size_t)t * nh + h) * vd + e] = __float2bfloat16_rn(o);
     }
 }
@@ -570,13 +561,13 @@ ST_EXPORT int st_gqa_attention_single(const void* q, const void* pool, long long
                                       const int* slots, const int* block_table, int max_pages, int n_tokens, int nh,
                                       int nkv, int dim, int vd, int page_size, float scale, int window, int keep_first,
                                       int has_sink, float sink, const void* gate, long long gate_ld, float out_scale,
-                                      int* status, void* stream, const float* sinks) {
+                                      int* status, void* stream, const float* sinks, int gate_heads) {
     if (n_tokens <= 0) return 0;
     if (page_size <= 0 || keep_first < 0) return ST_ERR_BAD_ARG;
     if (!st_gqa_attention_single_applies(nh, nkv, dim, vd)) return ST_ERR_BAD_SIZE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
     const GqaMask mask = {window, keep_first};
-    const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr};
+    const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr, gate_heads};
     cudaStream_t s = (cudaStream_t)stream;
     // Query heads per block: the whole group when that gives blocks for three quarters of the device (a key or value
     // row is then fetched once for the group), else the largest part of the group that does, down to one head; the

@@ -25,13 +25,15 @@ __device__ __forceinline__ bool gqa_seen(int key, int pos, const GqaMask& m) {
 }
 
 // What is done to a head's result before it is stored: times out_scale, and, with gate, times
-// sigmoid(gate[token * gate_ld + head * vd + e]) (gate logits as a product left them, in the storage type).
+// sigmoid(gate[token * gate_ld + head * vd + e]) (gate logits as a product left them, in the storage type), or, with
+// gate_heads, times sigmoid(gate[token * gate_ld + head]): one number for the whole head.
 // sinks: with has_sink, the extra term's logit of every head (float [heads]); null: the one `sink` for all heads.
 struct GqaEpilogue {
     const void* gate;
     long long gate_ld;
     float out_scale;
     const float* sinks;
+    int gate_heads;
 };
 
 __device__ __forceinline__ float sigmoidf_(float z) { return 1.f / (1.f + expf(-z)); }

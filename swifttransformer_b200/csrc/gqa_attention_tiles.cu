@@ -259,7 +259,8 @@ gqa_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__ 
         if (!live[r]) continue;
         const size_t t = (size_t)(first + off + row0 + g + 8 * r);
         bf16* orow = out + (t * nh + h) * vd;
-        const bf16* grow = gate ? gate + t * epi.gate_ld + (size_t)h * vd : nullptr;
+        const bf16* grow = gate && !epi.gate_heads ? gate + t * epi.gate_ld + (size_t)h * vd : nullptr;
+        if (gate && epi.gate_heads) inv[r] *= sigmoidf_(to_f32(gate[t * epi.gate_ld + h]));
 #pragma unroll
         for (int nt = 0; nt < VDT / 8; ++nt) {
             const int e = nt * 8 + 2 * tq;
@@ -300,20 +301,21 @@ ST_EXPORT int st_gqa_attention_tiles_applies(int dim, int vd) {
 
 // tiles: int32 [n_tiles][2] = (request of the step, offset of a tile of `tile_rows` query rows among its new tokens);
 // a tile whose offset lies past the request's tokens is padding.  gate: bfloat16 logits, the head's at
-// gate[token * gate_ld + head * vd ...], or null; gate_ld even and the pointer 4-byte aligned.
+// gate[token * gate_ld + head * vd ...], or null; gate_ld even and the pointer 4-byte aligned (not with gate_heads: one
+// logit per head at gate[token * gate_ld + head]).
 ST_EXPORT int st_gqa_attention_tiles(const void* q, const void* pool, long long page_stride, long long entry_offset,
                                      void* out, const int* tiles, int n_tiles, int tile_rows, const int* q_start,
                                      const int* start_pos, const int* slots, const int* block_table, int max_pages,
                                      int nh, int nkv, int dim, int vd, int page_size, float scale, int window,
                                      int keep_first, int has_sink, float sink, const void* gate, long long gate_ld,
-                                     float out_scale, int* status, void* stream, const float* sinks) {
+                                     float out_scale, int* status, void* stream, const float* sinks, int gate_heads) {
     if (n_tiles <= 0) return 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || tile_rows <= 0 || keep_first < 0) return ST_ERR_BAD_ARG;
     if (!st_gqa_attention_tiles_applies(dim, vd)) return ST_ERR_BAD_SIZE;
-    if (gate && ((gate_ld & 1) || ((uintptr_t)gate & 3))) return ST_ERR_BAD_ARG;
+    if (gate && !gate_heads && ((gate_ld & 1) || ((uintptr_t)gate & 3))) return ST_ERR_BAD_ARG;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
     const GqaMask mask = {window, keep_first};
-    const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr};
+    const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr, gate_heads};
     cudaStream_t s = (cudaStream_t)stream;
 #define GT_ARGS q, pool, c, out, tiles, n_tiles, tile_rows, q_start, start_pos, slots, block_table, nh, scale, mask, has_sink, \
                 sink, epi, status, s

@@ -5,13 +5,14 @@
 // v_h = Uv_h c); the kernels here work in the latent space: the query of head h arrives already multiplied by
 // Uk_h^T (kr numbers) followed by its own rotated part, so that
 //
-//   s_j   = scale * (q_lat . c_j + q_rot . k_rot_j)                  over the keys j <= the query's position
+//   s_j   = scale * (q_lat . c_j + q_rot . k_rot_j)                  over the keys j <= the query's position (with a
+//                                                                     window: the last `window` of them)
 //   p     = exp(s_j - m) / (sum_j exp(s_j - m) + exp(sink_h - m))    the sink has no key and no value
 //   o_lat = gate * sum_j p_j c_j                                     gate = sigmoid of the head's gate logit
 //
 // and head h's result is Uv_h o_lat, a product the caller does for all tokens at once.
 //
-// latent_prepare:  from the fused projection [dq | dkv | gates] of the step's tokens: RMS norm of the query latent
+// latent_prepare:  from the fused projection [dq | dkv | ...] of the step's tokens: RMS norm of the query latent, if there is one
 //                  (out, in the activation type), RMS norm of the key/value latent and rotation of the shared key
 //                  part by position, both written to the token's page.
 // latent_q_rotate: rotation of every head's rotated query part into the latent-space query rows.
@@ -19,16 +20,16 @@
 //                  aligned to absolute positions: a row's result does not depend on how the request was cut
 //                  into steps or on what else is in the batch.
 //
-// Rotation ("halves" layout): of the first rot_dims dimensions, i is paired with i + rot_dims/2 and the pair
-// (u, v) at position p becomes (u cos a - v sin a, v cos a + u sin a), a = p * inv_freq[i], angle in float.
+// Rotation (struct Rotation): halves or neighbours, the pair (u, v) at position p becomes
+// (u cos a - v sin a, v cos a + u sin a) times an amplitude, a = p * freq[i], angle in float.
 #include "latent_attention.cuh"
 
 #define LP_THREADS 128
 
 template <typename T>
 __global__ void __launch_bounds__(LP_THREADS)
-latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_rank, const float* __restrict__ q_w,
-                      const float* __restrict__ kv_w, float eps, const float* __restrict__ inv_freq, int rot_dims,
+latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_rank, int kv_off, const float* __restrict__ q_w,
+                      const float* __restrict__ kv_w, float eps, Rotation turn,
                       T* __restrict__ cq, T* __restrict__ pool, LatentCache cache, const int* __restrict__ positions,
                       const int* __restrict__ seq_of_token, const int* __restrict__ slots,
                       const int* __restrict__ block_table, int write_kv, int* __restrict__ status) {
@@ -41,16 +42,18 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_rank, const floa
     const T* row = proj + (size_t)t * ld;
     const int kr = cache.kr, rot = cache.rot;
     float ss = 0.f;
-    for (int e = threadIdx.x; e < q_rank; e += LP_THREADS) {
-        const float v = load1_cg(row + e);
-        ss = fmaf(v, v, ss);
+    if (q_rank > 0) {
+        for (int e = threadIdx.x; e < q_rank; e += LP_THREADS) {
+            const float v = load1_cg(row + e);
+            ss = fmaf(v, v, ss);
+        }
+        ss = block_sum(ss, scratch);
+        const float rq = rsqrtf(ss / (float)q_rank + eps);
+        for (int e = threadIdx.x; e < q_rank; e += LP_THREADS)
+            cq[(size_t)t * q_rank + e] = from_f32<T>(load1_cg(row + e) * rq * q_w[e]);
     }
-    ss = block_sum(ss, scratch);
-    const float rq = rsqrtf(ss / (float)q_rank + eps);
-    for (int e = threadIdx.x; e < q_rank; e += LP_THREADS)
-        cq[(size_t)t * q_rank + e] = from_f32<T>(load1_cg(row + e) * rq * q_w[e]);
     if (!write_kv) return;
-    const T* kv = row + q_rank;
+    const T* kv = row + kv_off;
     ss = 0.f;
     for (int e = threadIdx.x; e < kr; e += LP_THREADS) {
         const float v = load1_cg(kv + e);
@@ -65,76 +68,67 @@ latent_prepare_kernel(const T* __restrict__ proj, int ld, int q_rank, const floa
     }
     T* dst = latent_row(pool, cache, page, pos % cache.page_size);
     for (int e = threadIdx.x; e < kr; e += LP_THREADS) dst[e] = from_f32<T>(load1_cg(kv + e) * rk * kv_w[e]);
-    const int half = rot_dims / 2;
-    for (int i = threadIdx.x; i < half; i += LP_THREADS) {
-        float sn, cs;
-        sincosf((float)pos * inv_freq[i], &sn, &cs);
-        const float u = load1_cg(kv + kr + i), v = load1_cg(kv + kr + i + half);
-        dst[kr + i] = from_f32<T>(u * cs - v * sn);
-        dst[kr + i + half] = from_f32<T>(v * cs + u * sn);
+    for (int e = threadIdx.x; e < rot; e += LP_THREADS) {
+        float v = load1_cg(kv + kr + e);
+        if (e < turn.dims) v = rot_apply(turn, e, pos, v, load1_cg(kv + kr + rot_partner(turn, e)));
+        dst[kr + e] = from_f32<T>(v);
     }
-    for (int e = rot_dims + threadIdx.x; e < rot; e += LP_THREADS) dst[kr + e] = kv[kr + e];
 }
 
-ST_EXPORT int st_latent_prepare(const void* proj, int ld, int q_rank, const float* q_w, const float* kv_w, float eps,
-                                const float* inv_freq, int rot_dims, void* cq, void* pool, long long page_stride,
+// q_rank 0: there is no query latent (cq and q_w are not used); kv_off: the column of proj at which the latent begins
+ST_EXPORT int st_latent_prepare(const void* proj, int ld, int q_rank, int kv_off, const float* q_w, const float* kv_w, float eps,
+                                const float* inv_freq, int rot_dims, int neighbours, float rot_amp, void* cq, void* pool, long long page_stride,
                                 long long entry_offset, const int* positions, const int* seq_of_token,
                                 const int* slots, const int* block_table, int max_pages, int n_tokens, int kr, int rot,
                                 int page_size, int write_kv, int* status, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (q_rank <= 0 || kr <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || rot_dims % 2) return ST_ERR_BAD_SIZE;
+    if (q_rank < 0 || kv_off < 0 || kr <= 0 || rot < 0 || rot_dims < 0 || rot_dims > rot || rot_dims % 2) return ST_ERR_BAD_SIZE;
     LatentCache c{max_pages, page_size, kr, rot, page_stride, entry_offset};
+    const Rotation turn{inv_freq, rot_dims, neighbours, rot_amp};
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == 0)
         return st_launch_pdl("latent_prepare", latent_prepare_kernel<float>, dim3(n_tokens), dim3(LP_THREADS), 0, s,
-                             (const float*)proj, ld, q_rank, q_w, kv_w, eps, inv_freq, rot_dims, (float*)cq, (float*)pool,
+                             (const float*)proj, ld, q_rank, kv_off, q_w, kv_w, eps, turn, (float*)cq, (float*)pool,
                              c, positions, seq_of_token, slots, block_table, write_kv, status);
     if (dtype == 1)
         return st_launch_pdl("latent_prepare", latent_prepare_kernel<bf16>, dim3(n_tokens), dim3(LP_THREADS), 0, s,
-                             (const bf16*)proj, ld, q_rank, q_w, kv_w, eps, inv_freq, rot_dims, (bf16*)cq, (bf16*)pool, c,
+                             (const bf16*)proj, ld, q_rank, kv_off, q_w, kv_w, eps, turn, (bf16*)cq, (bf16*)pool, c,
                              positions, seq_of_token, slots, block_table, write_kv, status);
     return ST_ERR_BAD_DTYPE;
 }
 
-// q: [tokens, nh * (dim + rot)] as the up-projection left it; q_lat: [tokens, nh, kr + rot], whose last `rot`
+// q: [tokens, ld], the first nh * (dim + rot) columns as a projection left them; q_lat: [tokens, nh, kr + rot], whose last `rot`
 // numbers per head this kernel writes (the first kr are the product of the head's unrotated part with Uk_h).
 template <typename T>
 __global__ void __launch_bounds__(LP_THREADS)
-latent_q_rotate_kernel(const T* __restrict__ q, T* __restrict__ q_lat, const int* __restrict__ positions,
-                       const float* __restrict__ inv_freq, int rot_dims, int nh, int dim, int rot, int kr) {
+latent_q_rotate_kernel(const T* __restrict__ q, int ld, T* __restrict__ q_lat, const int* __restrict__ positions,
+                       Rotation turn, int nh, int dim, int rot, int kr) {
     ST_PDL_WAIT();
     ST_PDL_TRIGGER();
     const int t = blockIdx.x;
     const int pos = positions[t];
     if (pos < 0) return;
-    const int half = rot_dims / 2, per = half + (rot - rot_dims);
-    for (int i = threadIdx.x; i < nh * per; i += LP_THREADS) {
-        const int h = i / per, j = i % per;
-        const T* src = q + ((size_t)t * nh + h) * (dim + rot) + dim;
-        T* dst = q_lat + ((size_t)t * nh + h) * (kr + rot) + kr;
-        if (j < half) {
-            float sn, cs;
-            sincosf((float)pos * inv_freq[j], &sn, &cs);
-            const float u = load1_cg(src + j), v = load1_cg(src + j + half);
-            dst[j] = from_f32<T>(u * cs - v * sn);
-            dst[j + half] = from_f32<T>(v * cs + u * sn);
-        } else {
-            dst[rot_dims + j - half] = src[rot_dims + j - half];
-        }
+    for (int i = threadIdx.x; i < nh * rot; i += LP_THREADS) {
+        const int h = i / rot, e = i % rot;
+        const T* src = q + (size_t)t * ld + (size_t)h * (dim + rot) + dim;
+        float v = load1_cg(src + e);
+        if (e < turn.dims) v = rot_apply(turn, e, pos, v, load1_cg(src + rot_partner(turn, e)));
+        q_lat[((size_t)t * nh + h) * (kr + rot) + kr + e] = from_f32<T>(v);
     }
 }
 
-ST_EXPORT int st_latent_q_rotate(const void* q, void* q_lat, const int* positions, const float* inv_freq, int rot_dims,
-                                 int n_tokens, int nh, int dim, int rot, int kr, int dtype, void* stream) {
+ST_EXPORT int st_latent_q_rotate(const void* q, int ld, void* q_lat, const int* positions, const float* inv_freq,
+                                 int rot_dims, int neighbours, float rot_amp, int n_tokens, int nh, int dim, int rot, int kr, int dtype, void* stream) {
     if (n_tokens <= 0 || rot <= 0) return 0;
     if (rot_dims < 0 || rot_dims > rot || rot_dims % 2) return ST_ERR_BAD_SIZE;
+    const Rotation turn{inv_freq, rot_dims, neighbours, rot_amp};
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == 0)
         return st_launch_pdl("latent_q_rotate", latent_q_rotate_kernel<float>, dim3(n_tokens), dim3(LP_THREADS), 0, s,
-                             (const float*)q, (float*)q_lat, positions, inv_freq, rot_dims, nh, dim, rot, kr);
+                             (const float*)q, ld, (float*)q_lat, positions, turn, nh, dim, rot, kr);
     if (dtype == 1)
         return st_launch_pdl("latent_q_rotate", latent_q_rotate_kernel<bf16>, dim3(n_tokens), dim3(LP_THREADS), 0, s,
-                             (const bf16*)q, (bf16*)q_lat, positions, inv_freq, rot_dims, nh, dim, rot, kr);
+                             (const bf16*)q, ld, (bf16*)q_lat, positions, turn, nh, dim, rot, kr);
     return ST_ERR_BAD_DTYPE;
 }
 
@@ -148,7 +142,8 @@ latent_attention_plain_kernel(const T* __restrict__ q_lat, const T* __restrict__
                               T* __restrict__ out, const int* __restrict__ items, const int* __restrict__ positions,
                               const int* __restrict__ seq_of_token, const int* __restrict__ slots,
                               const int* __restrict__ block_table, const float* __restrict__ sink,
-                              const T* __restrict__ gates, int gate_ld, int nh, float scale, int* __restrict__ status) {
+                              const T* __restrict__ gates, int gate_ld, int nh, float scale, int window,
+                              int* __restrict__ status) {
     extern __shared__ float smem[];
     float* sq = smem;                       // [kr + rot]
     float* sp = smem + cache.kr + cache.rot;  // [LKT]
@@ -169,11 +164,11 @@ latent_attention_plain_kernel(const T* __restrict__ q_lat, const T* __restrict__
 #pragma unroll
     for (int c = 0; c < LVMAX; ++c) acc[c] = 0.f;
     float m = -INFINITY, l = 0.f;
-    const int hi = pos + 1;
-    for (int base = 0; base < hi; base += LKT) {
+    const int hi = pos + 1, lo = window > 0 ? max(0, hi - window) : 0;
+    for (int base = lo / LKT * LKT; base < hi; base += LKT) {      // (tiles aligned to absolute positions)
         const int j = base + threadIdx.x;
         float sc = -INFINITY;
-        if (j < hi) {
+        if (j >= lo && j < hi) {
             const int page = bt[j / ps];
             if (page >= 0) {
                 const T* krow = latent_row(pool, cache, page, j % ps);
@@ -191,13 +186,13 @@ latent_attention_plain_kernel(const T* __restrict__ q_lat, const T* __restrict__
         m = n;
         sp[threadIdx.x] = p;
         __syncthreads();
-        const int j_end = min(LKT, hi - base);
+        const int j_begin = max(0, lo - base), j_end = min(LKT, hi - base);
 #pragma unroll
         for (int c = 0; c < LVMAX; ++c) {
             const int e = threadIdx.x + c * LKT;
             if (e >= kr) continue;
             float x = acc[c] * corr;
-            for (int jj = 0; jj < j_end; ++jj) {
+            for (int jj = j_begin; jj < j_end; ++jj) {
                 const int key = base + jj;
                 const int page = bt[key / ps];
                 if (page < 0) continue;
@@ -227,7 +222,7 @@ ST_EXPORT int st_latent_attention_plain(const void* q_lat, const void* pool, lon
                                         void* out, const int* items, const int* positions, const int* seq_of_token,
                                         const int* slots, const int* block_table, int max_pages, int n_tokens, int nh,
                                         int kr, int rot, int page_size, const float* sink, const void* gates, int gate_ld,
-                                        float scale, int* status, int dtype, void* stream) {
+                                        float scale, int* status, int dtype, void* stream, int window) {
     if (n_tokens <= 0) return 0;
     if (kr <= 0 || rot < 0 || nh <= 0) return ST_ERR_BAD_SIZE;
     if (kr > LKT * LVMAX || nh > 65535) return ST_ERR_TOO_LARGE;
@@ -238,10 +233,10 @@ ST_EXPORT int st_latent_attention_plain(const void* q_lat, const void* pool, lon
     if (dtype == 0)
         return st_launch_pdl("latent_plain", latent_attention_plain_kernel<float>, grid, dim3(LKT), smem, s,
                              (const float*)q_lat, (const float*)pool, c, (float*)out, items, positions, seq_of_token, slots,
-                             block_table, sink, (const float*)gates, gate_ld, nh, scale, status);
+                             block_table, sink, (const float*)gates, gate_ld, nh, scale, window, status);
     if (dtype == 1)
         return st_launch_pdl("latent_plain", latent_attention_plain_kernel<bf16>, grid, dim3(LKT), smem, s,
                              (const bf16*)q_lat, (const bf16*)pool, c, (bf16*)out, items, positions, seq_of_token, slots,
-                             block_table, sink, (const bf16*)gates, gate_ld, nh, scale, status);
+                             block_table, sink, (const bf16*)gates, gate_ld, nh, scale, window, status);
     return ST_ERR_BAD_DTYPE;
 }

@@ -41,7 +41,7 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restri
                             bf16* __restrict__ out, const int* __restrict__ positions, const int* __restrict__ q_start,
                             const int* __restrict__ start_pos, const int* __restrict__ slots,
                             const int* __restrict__ block_table, int n_seqs, const float* __restrict__ sink,
-                            const bf16* __restrict__ gates, int gate_ld, int nh, float scale_log2, int lds, int kdp,
+                            const bf16* __restrict__ gates, int gate_ld, int nh, float scale_log2, int window, int lds, int kdp,
                             int n_splits, float* __restrict__ partial, int* __restrict__ status) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                 // [64][lds]
@@ -84,7 +84,8 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restri
     const int start = start_pos[b];
     const int* bt = block_table + (size_t)slots[b] * cache.max_pages;
     const int last_row = min(r0 + LM_ROWS, n_rows) - 1;
-    const int hi = start + last_row / nh + 1;           // keys 0 .. hi-1 are seen by some row of the tile
+    const int hi = start + last_row / nh + 1;           // keys lo .. hi-1 are seen by some row of the tile
+    const int lo = window > 0 ? max(0, start + r0 / nh - window + 1) : 0;
     const int chunks = kd / 8;
 
     // the queries: the tile's rows are consecutive in memory
@@ -97,13 +98,13 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restri
         }
     }
     // The key rows of a tile arrive as bulk copies, one per row, issued by the lanes of warp 0 (a lane per key: the 32
-    // page look-ups go out together) and completing on the stage's mbarrier; rows past the tile's last key keep what
+    // page look-ups go out together) and completing on the stage's mbarrier; rows outside the tile's key range keep what
     // an earlier tile left there (finite numbers, and every weight on them is zero).
     const uint32_t row_bytes = (uint32_t)kd * sizeof(bf16);
     auto load_keys = [&](int kt, int stage) {
         if (warp != 0) return;
         const int j = kt * LM_KEYS + lane;
-        bool ok = j < hi;
+        bool ok = j >= lo && j < hi;                    // (the pages before a window may be gone)
         const bf16* src = pool;
         if (ok) {
             const int page = bt[j / ps];
@@ -117,9 +118,9 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restri
         if (ok) bulk_row_copy(smem_u32(sK + (stage * LM_KEYS + lane) * lds), src, row_bytes, bar);
     };
     // the tile's key range, cut over blockIdx.y into parts of whole key tiles
-    const int all_kt = (hi + LM_KEYS - 1) / LM_KEYS;
-    const int per = (all_kt + n_splits - 1) / n_splits;
-    const int kt_begin = blockIdx.y * per, n_kt = min(all_kt, kt_begin + per);
+    const int all_kt = (hi + LM_KEYS - 1) / LM_KEYS, first_kt = lo / LM_KEYS;
+    const int per = (all_kt - first_kt + n_splits - 1) / n_splits;
+    const int kt_begin = first_kt + blockIdx.y * per, n_kt = min(all_kt, kt_begin + per);
     if (kt_begin < n_kt) load_keys(kt_begin, 0);
     cp_async_commit();
 
@@ -185,7 +186,8 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restri
             for (int e = 0; e < 4; ++e) {
                 const int j = kt * LM_KEYS + half * KW + nt * 8 + 2 * tq + (e & 1);
                 const int limit = e < 2 ? pos_a : pos_b;
-                const float v = j <= limit ? s[nt][e] * scale_log2 : -INFINITY;
+                const bool seen = j <= limit && (window <= 0 || limit - j < window);
+                const float v = seen ? s[nt][e] * scale_log2 : -INFINITY;
                 s[nt][e] = v;
                 mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }
@@ -210,7 +212,7 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restri
             // maximum has grown by more than LM_LAZY (in powers of two), so that the accumulator is rarely rescaled;
             // weights stay below 2^LM_LAZY, and the reference cancels in the end like a maximum does
             if (m[i] == -INFINITY) {
-                corr[i] = 1.f;                 // nothing accumulated yet
+                corr[i] = 1.f;                 // nothing accumulated yet (no key seen so far)
                 m[i] = mn;
             } else if (mn > m[i] + LM_LAZY) {
                 corr[i] = fast_exp2(m[i] - mn);
@@ -417,9 +419,10 @@ static long long lm_tiles(int n_tokens, int n_seqs, int nh) {
 // Into how many parts the key ranges of a step of this shape are cut: one when the tiles fill the device by
 // themselves (prompt portions), else as many as bring the launch to about a block per SM, 16 at most.  It depends on
 // the step's shape only (never on lengths), so a recorded step keeps it.
-ST_EXPORT int st_latent_attention_mma_splits(int n_tokens, int n_seqs, int nh) {
+ST_EXPORT int st_latent_attention_mma_splits(int n_tokens, int n_seqs, int nh, int window) {
     const long long tiles = lm_tiles(n_tokens, n_seqs, nh);
     long long n = st_sm_count() / (tiles > 0 ? tiles : 1);
+    if (window > 0 && n > window / LM_KEYS + 2) n = window / LM_KEYS + 2;      // a window spans no more key tiles
     return (int)(n < 1 ? 1 : n > 16 ? 16 : n);
 }
 
@@ -433,7 +436,8 @@ ST_EXPORT int st_latent_attention_mma(const void* q_lat, const void* pool, long 
                                       void* out, const int* positions, const int* q_start, const int* start_pos,
                                       const int* slots, const int* block_table, int max_pages, int n_tokens, int n_seqs,
                                       int nh, int kr, int rot, int page_size, const float* sink, const void* gates,
-                                      int gate_ld, float scale, int n_splits, float* partial, int* status, void* stream) {
+                                      int gate_ld, float scale, int n_splits, float* partial, int* status, void* stream,
+                                      int window) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (!st_latent_attention_mma_applies(kr, rot) || page_stride % 8 || entry_offset % 8) return ST_ERR_BAD_SIZE;
     if (!aligned16(q_lat) || !aligned16(pool) || n_splits < 1 || n_splits > 64 || (n_splits > 1 && !partial)) return ST_ERR_BAD_ARG;
@@ -454,7 +458,7 @@ ST_EXPORT int st_latent_attention_mma(const void* q_lat, const void* pool, long 
         }                                                                                                            \
         rc = st_launch_pdl("latent_mma", latent_attention_mma_kernel<NTV, NPV>, dim3((unsigned)tiles, n_splits), dim3(NPV * 128), \
                            smem, s, (const bf16*)q_lat, (const bf16*)pool, c, (bf16*)out, positions, q_start, start_pos,  \
-                           slots, block_table, n_seqs, sink, (const bf16*)gates, gate_ld, nh, scale_log2, lds, kdp,      \
+                           slots, block_table, n_seqs, sink, (const bf16*)gates, gate_ld, nh, scale_log2, window, lds, kdp,      \
                            n_splits, partial, status);                                                               \
     }
     LM_LAUNCH(2, 2) LM_LAUNCH(4, 2) LM_LAUNCH(6, 2) LM_LAUNCH(8, 2)

@@ -4,6 +4,10 @@
 // moe_route:   z = W_r h (float, W_r float [experts, width]); s = softmax(z) over all experts; the `top` experts
 //              with the largest s (ties: the lower index) and their s as weights (not renormalised, unless asked: then divided by their sum + 1e-20);
 //              optionally g = sigmoid(w_g . h), one number per token (the gate of a shared expert).
+//              RouteRule: scores may be sigmoid(z) instead; the experts may form equal groups of neighbours, of which
+//              only the `keep` best (by the sum of a group's two largest scores; ties: the lower index) can be chosen
+//              from; the weights are multiplied by `scale` in the end.  The logits may come from a product of their
+//              own (z float [tokens, ld]) instead of being formed here.
 //              A padding token (position < 0) gets expert -1.
 // moe_sort:    the step's (token, choice) items grouped by expert: offsets[e]..offsets[e+1] are expert e's places
 //              in `sorted` (item indices), `place[item]` the inverse, and a list of row tiles (expert, first place)
@@ -15,12 +19,83 @@
 #define ROUTE_THREADS 256
 #define ROUTE_MAX_EXPERTS 1024
 
+struct RouteRule {
+    int sigmoid, groups, keep, renorm;      // groups <= 1: no groups
+    float scale;
+};
+
+// The choice of one token by one warp from its logits z[0..n_experts) in shared memory (overwritten).
+__device__ __forceinline__ void route_choose(float* z, int n_experts, int top, const RouteRule& rule, int lane,
+                                             int* __restrict__ experts, float* __restrict__ weights) {
+    float inv = 1.f;
+    if (rule.sigmoid) {
+        for (int e = lane; e < n_experts; e += 32) z[e] = 1.f / (1.f + expf(-z[e]));
+    } else {
+        float m = -INFINITY;
+        for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, z[e]);
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int e = lane; e < n_experts; e += 32) {
+            const float p = expf(z[e] - m);
+            z[e] = p;
+            sum += p;
+        }
+        inv = 1.f / warp_sum(sum);
+    }
+    __syncwarp();
+    if (rule.groups > 1) {
+        // a lane per group (in turns of 32): the sum of its two largest scores; a group is kept when fewer than
+        // `keep` groups stand before it (a larger sum, or the same sum and a lower index)
+        const int per = n_experts / rule.groups;
+        float* gs = z + n_experts;
+        for (int g = lane; g < rule.groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;
+            for (int i = 0; i < per; ++i) {
+                const float v = z[g * per + i];
+                if (v > a) { b = a; a = v; } else if (v > b) b = v;
+            }
+            gs[g] = per > 1 ? a + b : a;
+        }
+        __syncwarp();
+        for (int g = lane; g < rule.groups; g += 32) {
+            int before = 0;
+            for (int o = 0; o < rule.groups; ++o) before += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
+            if (before >= rule.keep)
+                for (int i = 0; i < per; ++i) z[g * per + i] = -1.f;      // below every score, above a chosen one's mark
+        }
+        __syncwarp();
+    }
+    float chosen_sum = 0.f;
+    for (int k = 0; k < top; ++k) {
+        float best = -1.5f;
+        int arg = 0x7fffffff;
+        for (int e = lane; e < n_experts; e += 32)
+            if (z[e] > best) { best = z[e]; arg = e; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+            if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+        }
+        const float w = fmaxf(best, 0.f) * inv;      // (an expert outside the kept groups, if there are too few inside: weight 0)
+        chosen_sum += w;
+        if (lane == 0) {
+            experts[k] = arg;
+            weights[k] = w * (rule.renorm ? 1.f : rule.scale);
+            z[arg] = -2.f;
+        }
+        __syncwarp();
+    }
+    if (rule.renorm && lane == 0)
+        for (int k = 0; k < top; ++k) weights[k] = weights[k] / (chosen_sum + 1e-20f) * rule.scale;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const T* __restrict__ h, int width, const float* __restrict__ w_r, int n_experts, int top,
-                 int renorm, const float* __restrict__ w_g, const int* __restrict__ positions,
+                 RouteRule rule, const float* __restrict__ w_g, const int* __restrict__ positions,
                  int* __restrict__ experts, float* __restrict__ weights, float* __restrict__ gate, int vec) {
-    __shared__ float z[ROUTE_MAX_EXPERTS + 1];
+    extern __shared__ float z[];           // [n_experts + groups + 1]
     ST_PDL_WAIT();
     ST_PDL_TRIGGER();
     const int t = blockIdx.x;
@@ -45,61 +120,67 @@ moe_route_kernel(const T* __restrict__ h, int width, const float* __restrict__ w
             for (int i = lane; i < width; i += 32) d = fmaf(load1_cg(row + i), wr[i], d);
         }
         d = warp_sum(d);
-        if (lane == 0) z[e] = d;
+        if (lane == 0) z[e < n_experts ? e : n_experts + rule.groups] = d;
     }
     __syncthreads();
     if (warp != 0) return;
-    if (w_g && lane == 0) gate[t] = 1.f / (1.f + expf(-z[n_experts]));
-    float m = -INFINITY;
-    for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, z[e]);
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int e = lane; e < n_experts; e += 32) {
-        const float p = expf(z[e] - m);
-        z[e] = p;
-        sum += p;
-    }
-    sum = warp_sum(sum);
-    __syncwarp();
-    const float inv = 1.f / sum;
-    float chosen_sum = 0.f;
-    for (int k = 0; k < top; ++k) {
-        float best = -1.f;
-        int arg = 0x7fffffff;
-        for (int e = lane; e < n_experts; e += 32)
-            if (z[e] > best) { best = z[e]; arg = e; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-            if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-        }
-        chosen_sum += best * inv;
-        if (lane == 0) {
-            experts[(size_t)t * top + k] = arg;
-            weights[(size_t)t * top + k] = best * inv;
-            z[arg] = -2.f;
-        }
-        __syncwarp();
-    }
-    if (renorm && lane == 0)
-        for (int k = 0; k < top; ++k) weights[(size_t)t * top + k] /= chosen_sum + 1e-20f;
+    if (w_g && lane == 0) gate[t] = 1.f / (1.f + expf(-z[n_experts + rule.groups]));
+    route_choose(z, n_experts, top, rule, lane, experts + (size_t)t * top, weights + (size_t)t * top);
 }
 
-ST_EXPORT int st_moe_route(const void* h, int n_tokens, int width, const float* w_r, int n_experts, int top, int renorm,
-                           const float* w_g, const int* positions, int* experts, float* weights, float* gate, int dtype,
+// The choice alone, from logits a product left: a warp per token.
+#define CHOOSE_WARPS 4
+__global__ void __launch_bounds__(CHOOSE_WARPS * 32)
+moe_choose_kernel(const float* __restrict__ logits, int ld, int n_tokens, int n_experts, int top, RouteRule rule,
+                  const int* __restrict__ positions, int* __restrict__ experts, float* __restrict__ weights) {
+    extern __shared__ float z_all[];       // [CHOOSE_WARPS][n_experts + groups]
+    ST_PDL_WAIT();
+    ST_PDL_TRIGGER();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t = blockIdx.x * CHOOSE_WARPS + warp;
+    if (t >= n_tokens) return;
+    if (positions && positions[t] < 0) {
+        for (int k = lane; k < top; k += 32) { experts[(size_t)t * top + k] = -1; weights[(size_t)t * top + k] = 0.f; }
+        return;
+    }
+    float* z = z_all + warp * (n_experts + rule.groups);
+    for (int e = lane; e < n_experts; e += 32) z[e] = __ldcg(logits + (size_t)t * ld + e);
+    __syncwarp();
+    route_choose(z, n_experts, top, rule, lane, experts + (size_t)t * top, weights + (size_t)t * top);
+}
+
+static int route_rule_bad(const RouteRule& r, int n_experts, int top) {
+    if (n_experts <= 0 || top <= 0 || top > n_experts || r.groups < 0) return 1;
+    return r.groups > 1 && (n_experts % r.groups || r.keep <= 0 || r.keep > r.groups);
+}
+
+ST_EXPORT int st_moe_choose(const float* logits, int ld, int n_tokens, int n_experts, int top, int sigmoid, int groups,
+                            int keep, int renorm, float scale, const int* positions, int* experts, float* weights, void* stream) {
+    if (n_tokens <= 0) return 0;
+    const RouteRule rule{sigmoid, groups, keep, renorm, scale};
+    if (route_rule_bad(rule, n_experts, top) || ld < n_experts) return ST_ERR_BAD_ARG;
+    if (n_experts > ROUTE_MAX_EXPERTS) return ST_ERR_TOO_LARGE;
+    const size_t smem = (size_t)CHOOSE_WARPS * (n_experts + groups) * sizeof(float);
+    return st_launch_pdl("moe_choose", moe_choose_kernel, dim3((n_tokens + CHOOSE_WARPS - 1) / CHOOSE_WARPS), dim3(CHOOSE_WARPS * 32),
+                         smem, (cudaStream_t)stream, logits, ld, n_tokens, n_experts, top, rule, positions, experts, weights);
+}
+
+ST_EXPORT int st_moe_route(const void* h, int n_tokens, int width, const float* w_r, int n_experts, int top, int sigmoid,
+                           int groups, int keep, int renorm, float scale, const float* w_g, const int* positions, int* experts, float* weights, float* gate, int dtype,
                            void* stream) {
     if (n_tokens <= 0) return 0;
-    if (n_experts <= 0 || top <= 0 || top > n_experts) return ST_ERR_BAD_ARG;
+    const RouteRule rule{sigmoid, groups, keep, renorm, scale};
+    if (route_rule_bad(rule, n_experts, top)) return ST_ERR_BAD_ARG;
     if (n_experts > ROUTE_MAX_EXPERTS) return ST_ERR_TOO_LARGE;
     cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = (size_t)(n_experts + groups + 1) * sizeof(float);
     const int vec = width % 4 == 0 && aligned16(h) && aligned16(w_r) && (!w_g || aligned16(w_g));
     if (dtype == 0)
-        return st_launch_pdl("moe_route", moe_route_kernel<float>, dim3(n_tokens), dim3(ROUTE_THREADS), 0, s, (const float*)h,
-                             width, w_r, n_experts, top, renorm, w_g, positions, experts, weights, gate, vec);
+        return st_launch_pdl("moe_route", moe_route_kernel<float>, dim3(n_tokens), dim3(ROUTE_THREADS), smem, s, (const float*)h,
+                             width, w_r, n_experts, top, rule, w_g, positions, experts, weights, gate, vec);
     if (dtype == 1)
-        return st_launch_pdl("moe_route", moe_route_kernel<bf16>, dim3(n_tokens), dim3(ROUTE_THREADS), 0, s, (const bf16*)h,
-                             width, w_r, n_experts, top, renorm, w_g, positions, experts, weights, gate, vec);
+        return st_launch_pdl("moe_route", moe_route_kernel<bf16>, dim3(n_tokens), dim3(ROUTE_THREADS), smem, s, (const bf16*)h,
+                             width, w_r, n_experts, top, rule, w_g, positions, experts, weights, gate, vec);
     return ST_ERR_BAD_DTYPE;
 }
 

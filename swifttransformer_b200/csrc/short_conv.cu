@@ -4,6 +4,9 @@
 //
 //   y[t][c] = sum_j w[c][j] * u[t - taps + 1 + j][c]          (zeros before position 0)
 //
+// conv_residual: out = u + y (or y alone).  conv_act: out = act(y + b) from the first columns of a wider projection,
+// for mixers whose convolution stands inside.
+//
 // The state of a request holds the inputs at positions len-(taps-1) .. len-1
 // in that order (zero where the position is negative: a fresh slot is all
 // zeros, which is exactly "nothing before the sequence's start").
@@ -123,6 +126,116 @@ conv_state_update_kernel(const TI* __restrict__ in, int ld, float* __restrict__ 
         v[j] = src < keep ? st[(size_t)src * channels] : to_f32(in[(size_t)(first + src - keep) * ld + c]);
     }
     for (int j = 0; j < keep; ++j) st[(size_t)j * channels] = v[j];
+}
+
+// out[t][c] = act(bias[c] + conv(in)[t][c]);  in: [tokens, ld], its first `channels` columns.  A thread owns V
+// neighbouring channels of TT consecutive tokens of the step and carries the last taps - 1 inputs along in registers:
+// where a request begins (or the thread's first token lies inside one) they are fetched anew, from the step's own rows
+// and, before the step's first token of the request, from its state.  The state is read by several threads and stays
+// as it is (conv_state_update follows), unless `move_state` says that every request brings exactly one token: then the
+// one thread that reads a request's state for a channel also moves it on.
+template <typename T, int V, int TT>
+__global__ void __launch_bounds__(128)
+conv_act_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, const float* __restrict__ bias,
+                float* __restrict__ state, T* __restrict__ out, const int* __restrict__ positions,
+                const int* __restrict__ seq_of_token, const int* __restrict__ q_start, const int* __restrict__ slots,
+                int n_tokens, int channels, int taps, int act, int move_state) {
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    float wv[V][CONV_MAX_TAPS], bv[V];
+    if (c < channels) {                                 // no kernel writes the filters: fetched before the wait
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+            bv[v] = bias ? bias[c + v] : 0.f;
+#pragma unroll
+            for (int j = 0; j < CONV_MAX_TAPS; ++j)     // the newest input's weight stands last, whatever taps is
+                wv[v][j] = j >= CONV_MAX_TAPS - taps ? w[(size_t)(c + v) * taps + j - (CONV_MAX_TAPS - taps)] : 0.f;
+        }
+    }
+    ST_PDL_WAIT();
+    ST_PDL_TRIGGER();
+    if (c >= channels) return;
+    const int keep = taps - 1;
+    float u[CONV_MAX_TAPS][V];                          // u[CONV_MAX_TAPS - 1 - k]: the input k tokens back
+    int held = -1;                                      // the request whose inputs u holds
+    for (int k = 0; k < TT; ++k) {
+        const int t = blockIdx.x * TT + k;
+        if (t >= n_tokens) return;
+        if (positions[t] < 0) continue;                 // padding token of a fixed-shape step
+        const int b = seq_of_token[t];
+        float* st = state + (size_t)slots[b] * keep * channels + c;
+        if (b != held) {
+            held = b;
+            const int i = t - q_start[b];
+#pragma unroll
+            for (int j = 1; j < CONV_MAX_TAPS; ++j) {
+                float x[V];
+#pragma unroll
+                for (int v = 0; v < V; ++v) x[v] = 0.f;
+                if (j <= keep) {
+                    if (j <= i) load_v<V>(in + (size_t)(t - j) * ld + c, x);
+                    else load_v<V>(st + (size_t)(keep + i - j) * channels, x);
+                }
+#pragma unroll
+                for (int v = 0; v < V; ++v) u[CONV_MAX_TAPS - 1 - j][v] = x[v];
+            }
+        }
+        load_v<V>(in + (size_t)t * ld + c, u[CONV_MAX_TAPS - 1]);
+        float y[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+            y[v] = bv[v];
+#pragma unroll
+            for (int j = 0; j < CONV_MAX_TAPS; ++j) y[v] = fmaf(wv[v][j], u[j][v], y[v]);
+            y[v] = apply_act(y[v], act);
+        }
+        store_v<V>(out + (size_t)t * channels + c, y);
+        if (move_state) {
+#pragma unroll
+            for (int j = 0; j < CONV_MAX_TAPS - 1; ++j)          // the oldest kept input stands first
+                if (j < keep) {
+                    float x[V];
+#pragma unroll
+                    for (int v = 0; v < V; ++v) {
+                        x[v] = 0.f;
+#pragma unroll
+                        for (int q = 0; q < CONV_MAX_TAPS; ++q)
+                            if (q == CONV_MAX_TAPS - keep + j) x[v] = u[q][v];
+                    }
+                    store_v<V>(st + (size_t)j * channels, x);
+                }
+        }
+#pragma unroll
+        for (int j = 0; j + 1 < CONV_MAX_TAPS; ++j)
+#pragma unroll
+            for (int v = 0; v < V; ++v) u[j][v] = u[j + 1][v];
+    }
+}
+
+ST_EXPORT int st_conv_act(const void* in, int ld, const float* w, const float* bias, float* state, void* out,
+                          const int* positions, const int* seq_of_token, const int* q_start, const int* slots,
+                          int n_tokens, int channels, int taps, int act, int move_state, int dtype, void* stream) {
+    if (n_tokens <= 0) return 0;
+    if (channels <= 0 || taps < 1 || ld < channels || act < 0 || act > 5) return ST_ERR_BAD_ARG;
+    if (taps > CONV_MAX_TAPS) return ST_ERR_TOO_LARGE;
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool vec = channels % 4 == 0 && ld % 4 == 0 && aligned16(in) && aligned16(out) && aligned16(state);
+    const int per_block = vec ? 128 * 4 : 128;
+    const int tt = n_tokens > 256 ? 8 : 1;              // few tokens: a thread each; many: the inputs are fetched once
+    dim3 grid((n_tokens + tt - 1) / tt, (channels + per_block - 1) / per_block);
+#define CA_LAUNCH(T, V, TT)                                                                                              \
+    return st_launch_pdl("conv_act", conv_act_kernel<T, V, TT>, grid, dim3(128), 0, s, (const T*)in, ld, w, bias, state, \
+                         (T*)out, positions, seq_of_token, q_start, slots, n_tokens, channels, taps, act, move_state)
+#define CA_PICK(T)                                                                              \
+    do {                                                                                        \
+        if (vec) { if (tt == 8) CA_LAUNCH(T, 4, 8); CA_LAUNCH(T, 4, 1); }                       \
+        if (tt == 8) CA_LAUNCH(T, 1, 8);                                                        \
+        CA_LAUNCH(T, 1, 1);                                                                     \
+    } while (0)
+    if (dtype == 0) CA_PICK(float);
+    if (dtype == 1) CA_PICK(bf16);
+    return ST_ERR_BAD_DTYPE;
+#undef CA_PICK
+#undef CA_LAUNCH
 }
 
 // in: [n_tokens, channels] float (in_f32) or the storage type; out: [n_tokens, channels] storage type `dtype`

@@ -49,9 +49,11 @@ class ModelDef:
     # the most tokens a request may hold (the architecture's context length, from its configuration);
     # None: whatever the position encoding allows, and where that has no limit, the engine's own setting
     max_seq_len: Optional[int] = None
+    # parts that several blocks share (a table every layer reads)
+    shared_parts: List[Part] = dataclasses.field(default_factory=list)
 
     def parts(self) -> List[Part]:
-        out: List[Part] = [self.embedding, self.position]
+        out: List[Part] = [self.embedding, self.position] + list(self.shared_parts)
         for b in self.blocks:
             out.append(b)
         if self.final_norm is not None:

@@ -21,7 +21,7 @@ from . import build as _build
 
 _LIB = None
 
-ACT_CODES = {"none": 0, "relu": 1, "gelu": 2, "gelu_tanh": 3, "silu": 4}
+ACT_CODES = {"none": 0, "relu": 1, "gelu": 2, "gelu_tanh": 3, "silu": 4, "relu2": 5}
 NORM_CODES = {"layernorm": 0, "rmsnorm": 1, "none": 2}
 
 _ERRORS = {-1: "unsupported dtype", -2: "unsupported size", -3: "size beyond the kernel's limit",
@@ -725,12 +725,74 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, mult: float, 
                              _p(out_act), _dt(y), _stream()), "norm_add")
 
 
-def gated_act(gu: torch.Tensor, act: str) -> torch.Tensor:
-    """act(gu[:, :inner]) * gu[:, inner:] for the fused gate | up product gu [rows, 2 * inner]."""
-    assert gu.is_contiguous() and gu.shape[1] % 2 == 0
-    inner = gu.shape[1] // 2
+def conv_act(x: torch.Tensor, channels: int, w: torch.Tensor, bias: Optional[torch.Tensor], act: str, state: torch.Tensor,
+             positions: torch.Tensor, seq_of_token: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor,
+             move_state: bool = False) -> torch.Tensor:
+    """act(bias + sum_j w[:, j] * x[t - taps + 1 + j]) along each request's tokens for the first ``channels`` columns of
+    x [tokens, columns]; -> [tokens, channels] in x's type.  w float32 [channels, taps], bias float32 [channels] or None,
+    state float32 [slots, taps - 1, channels]: a request's last taps - 1 inputs, read; ``move_state``: only for steps in
+    which every request brings exactly one token, the kernel then moves the state on (else ``conv_state_update``
+    follows)."""
+    taps = w.shape[1]
+    assert x.is_contiguous() and x.shape[1] >= channels and w.dtype == torch.float32 and w.is_contiguous()
+    assert w.shape[0] == channels and state.dtype == torch.float32 and state.is_contiguous()
+    assert state.shape[1:] == (taps - 1, channels)
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == channels)
+    out = torch.empty((x.shape[0], channels), dtype=x.dtype, device=x.device)
+    _check(lib().st_conv_act(_p(x), x.shape[1], _p(w), _p(bias), _p(state), _p(out), _p(positions), _p(seq_of_token),
+                             _p(q_start), _p(slots), x.shape[0], channels, taps, ACT_CODES[act], int(move_state), _dt(x),
+                             _stream()), "conv_act")
+    return out
+
+
+def gated_norm_add(x: torch.Tensor, y: torch.Tensor, gate: Optional[torch.Tensor], gate_bias: Optional[torch.Tensor],
+                   gain: torch.Tensor, eps: float, positions: Optional[torch.Tensor] = None,
+                   next_gain: Optional[torch.Tensor] = None, next_eps: float = 0.0,
+                   out_act: Optional[torch.Tensor] = None) -> None:
+    """x[r] += gain * u / sqrt(mean(u^2) + eps) in place on the float32 residual rows, with u = y[r], or y[r] *
+    sigmoid(gate[r] + gate_bias) element by element (``gate``: logits [rows, width] in the activation type, any row
+    stride; ``gate_bias`` float32 [width]).  ``out_act``: also what reads x next, in the activation type: the new x,
+    RMS-normed with ``next_gain`` and ``next_eps`` if a gain is given.  Rows at a negative position are left alone."""
+    n, width = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and y.shape == x.shape
+    assert gain.dtype == torch.float32 and gain.numel() == width
+    low = out_act if out_act is not None else (gate if gate is not None else y)
+    assert y.dtype == torch.float32 or y.dtype == low.dtype
+    if gate is not None:
+        assert gate.shape == x.shape and gate.stride(1) == 1 and gate.dtype == low.dtype
+        assert gate_bias is not None and gate_bias.dtype == torch.float32 and gate_bias.numel() == width
+    if out_act is not None:
+        assert out_act.shape == x.shape and out_act.is_contiguous()
+    _check(lib().st_gated_norm_add(_p(x), _p(y), int(y.dtype == torch.float32), _p(gate),
+                                   gate.stride(0) if gate is not None else 0, _p(gate_bias), _p(gain), _f(eps),
+                                   _p(next_gain), _f(next_eps), n, width, _p(positions), _p(out_act), _dt(low), _stream()),
+           "gated_norm_add")
+
+
+def side_input(s: torch.Tensor, table: torch.Tensor, col0: int, ids: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(s[r]) * table[ids[r], col0 : col0 + dim] for float32 rows s [rows, dim]; -> the table's type."""
+    n, dim = s.shape
+    assert s.dtype == torch.float32 and s.is_contiguous() and table.is_contiguous() and ids.numel() == n
+    out = torch.empty((n, dim), dtype=table.dtype, device=s.device)
+    _check(lib().st_side_input(_p(s), _p(table), ctypes.c_longlong(table.shape[1]), col0, _p(ids), _p(out), n, dim,
+                               _dt(table), _stream()), "side_input")
+    return out
+
+
+def slice_rows(x: torch.Tensor, col0: int, cols: int, dtype: torch.dtype) -> torch.Tensor:
+    """Columns col0 .. col0 + cols - 1 of float32 rows, as a dense tensor of the given type."""
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    out = torch.empty((x.shape[0], cols), dtype=dtype, device=x.device)
+    _check(lib().st_slice_rows(_p(x), x.shape[1], col0, _p(out), x.shape[0], cols, _dt(out), _stream()), "slice_rows")
+    return out
+
+
+def gated_act(gu: torch.Tensor, act: str, inner: Optional[int] = None) -> torch.Tensor:
+    """act(gu[:, :inner]) * gu[:, inner : 2 * inner] for the fused gate | up product gu (``inner`` None: half its columns)."""
+    assert gu.is_contiguous() and (inner is not None or gu.shape[1] % 2 == 0)
+    inner = gu.shape[1] // 2 if inner is None else int(inner)
     out = torch.empty((gu.shape[0], inner), dtype=gu.dtype, device=gu.device)
-    _check(lib().st_gated_act(_p(gu), _p(out), gu.shape[0], inner, ACT_CODES[act], _dt(gu), _stream()), "gated_act")
+    _check(lib().st_gated_act(_p(gu), gu.shape[1], _p(out), gu.shape[0], inner, ACT_CODES[act], _dt(gu), _stream()), "gated_act")
     return out
 
 
@@ -857,6 +919,64 @@ def hgrn2_scan(proj: torch.Tensor, q_off: int, f_off: int, v_off: int, f_bias: t
     return out
 
 
+# ------------------------------------------------------------ the selective scan
+MAMBA_CHUNK = 64        # tokens of a chunk: longer portions are scanned in chunks side by side
+
+
+def mamba_scan_scratch(n_chunks: int, inner: int, n: int) -> int:
+    """Floats of scratch ``mamba_scan`` needs with that many chunks."""
+    return n_chunks * inner * (n + 1)
+
+
+def mamba_scan(x: torch.Tensor, dt: torch.Tensor, xd: torch.Tensor, b_off: int, c_off: int, proj: torch.Tensor, z_off: int,
+               A: torch.Tensor, D: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+               positions: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, n_seqs: int, write_state: bool = True,
+               chunks: Optional[torch.Tensor] = None, chunk_first: Optional[torch.Tensor] = None, n_chunks: int = 0,
+               chunk: int = 0, scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The selective scan over each request's tokens of the step: d = softplus(dt + dt_bias);
+    S <- exp(d A) S + d x B^T;  y = S C + D x;  out = y * silu(z).  x [tokens, inner] and ``proj`` [tokens, columns] (z at
+    column z_off) in the activation type; dt float32 [tokens, inner] (overwritten); xd float32 [tokens, columns] with B at
+    b_off and C at c_off; A [inner, n] (negative), D, dt_bias [inner] float32; state float32 [slots, inner, n].
+    ``chunks`` int32 [n_chunks, 2] = (request, offset), ``chunk_first`` [n_seqs + 1], ``chunk`` tokens each, ``scratch``
+    (``mamba_scan_scratch`` floats): long portions in chunks side by side; None: one run per request."""
+    tokens, inner = x.shape
+    n = A.shape[1]
+    assert x.is_contiguous() and out.is_contiguous() and out.shape == x.shape and out.dtype == x.dtype == proj.dtype
+    assert dt.dtype == xd.dtype == torch.float32 and dt.is_contiguous() and dt.shape == x.shape and xd.is_contiguous()
+    assert proj.is_contiguous() and proj.shape[1] >= z_off + inner and A.is_contiguous() and A.shape[0] == inner
+    assert A.dtype == D.dtype == dt_bias.dtype == torch.float32 and D.numel() == dt_bias.numel() == inner
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (inner, n)
+    buf = sums = None
+    if chunks is not None:
+        assert scratch is not None and scratch.numel() >= mamba_scan_scratch(n_chunks, inner, n)
+        buf, sums = scratch, scratch[n_chunks * inner * n:]
+    z = ctypes.c_void_p(proj.data_ptr() + z_off * proj.element_size())
+    _check(lib().st_mamba_scan(_p(x), _p(dt), _p(xd), xd.shape[1], b_off, c_off, z, proj.shape[1], _p(out), _p(A), _p(D),
+                               _p(dt_bias), _p(state), int(write_state), _p(buf), _p(sums), _p(positions), _p(q_start),
+                               _p(slots), n_seqs, _p(chunks), _p(chunk_first), n_chunks, chunk, inner, n, _dt(x),
+                               _stream()), "mamba_scan")
+    return out
+
+
+def mamba_single(x: torch.Tensor, xd: torch.Tensor, b_off: int, c_off: int, w_dt: torch.Tensor, proj: torch.Tensor,
+                 z_off: int, A: torch.Tensor, D: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor,
+                 out: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor, slots: torch.Tensor,
+                 write_state: bool = True) -> torch.Tensor:
+    """``mamba_scan`` for steps in which every request brings one token, with the product dt = xd[:, :rank] w_dt^T in the
+    same kernel; w_dt [inner, rank] (rank a multiple of 8) in the activation type."""
+    tokens, inner = x.shape
+    n, rank = A.shape[1], w_dt.shape[1]
+    assert x.is_contiguous() and out.is_contiguous() and out.shape == x.shape and out.dtype == x.dtype == proj.dtype
+    assert xd.dtype == torch.float32 and xd.is_contiguous() and w_dt.is_contiguous() and w_dt.dtype == x.dtype
+    assert proj.is_contiguous() and proj.shape[1] >= z_off + inner and A.is_contiguous() and A.shape[0] == inner
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (inner, n)
+    z = ctypes.c_void_p(proj.data_ptr() + z_off * proj.element_size())
+    _check(lib().st_mamba_single(_p(x), _p(xd), xd.shape[1], rank, b_off, c_off, _p(w_dt), z, proj.shape[1], _p(out), _p(A),
+                                 _p(D), _p(dt_bias), _p(state), int(write_state), _p(positions), _p(seq_of_token),
+                                 _p(slots), tokens, inner, n, _dt(x), _stream()), "mamba_single")
+    return out
+
+
 # ------------------------------------------------------------ latent attention
 def _latent_pool(pool: torch.Tensor, layer: int, kr: int, rot: int, page_size: int):
     """(page stride, offset of the entry) in elements, for a pool [pages, entries, page_size * (kr + rot)]."""
@@ -865,29 +985,36 @@ def _latent_pool(pool: torch.Tensor, layer: int, kr: int, rot: int, page_size: i
 
 
 def latent_prepare(proj: torch.Tensor, q_rank: int, q_norm: torch.Tensor, kv_norm: torch.Tensor, eps: float,
-                   inv_freq: torch.Tensor, rot_dims: int, cq: torch.Tensor, pool: torch.Tensor, layer: int,
+                   inv_freq: torch.Tensor, rot_dims: int, cq: Optional[torch.Tensor], pool: torch.Tensor, layer: int,
                    positions: torch.Tensor, seq_of_token: torch.Tensor, slots: torch.Tensor, block_table: torch.Tensor,
-                   kr: int, rot: int, page_size: int, status: torch.Tensor, write_kv: bool = True) -> None:
+                   kr: int, rot: int, page_size: int, status: torch.Tensor, write_kv: bool = True,
+                   kv_off: Optional[int] = None, neighbours: bool = False, rot_amp: float = 1.0) -> None:
     """From the fused projection [query latent (q_rank) | key/value latent (kr) | shared key part (rot) | ...] of the
     step's tokens: cq = the query latent, RMS-normed with ``q_norm``; the key/value latent RMS-normed with ``kv_norm``
-    and the shared key part, its first ``rot_dims`` dimensions rotated in halves by position * inv_freq, go to the
-    token's row of its page.  Statistics and angles are float."""
-    assert proj.is_contiguous() and proj.shape[1] >= q_rank + kr + rot and cq.shape == (proj.shape[0], q_rank)
-    assert cq.is_contiguous() and pool.dtype == proj.dtype == cq.dtype
+    and the shared key part, its first ``rot_dims`` dimensions rotated by position * inv_freq (in halves, or in pairs of
+    ``neighbours``; sine and cosine times ``rot_amp``), go to the token's row of its page.  Statistics and angles are
+    float.  ``q_rank`` 0 (cq and q_norm None): no query latent.  ``kv_off``: the column at which the key/value latent
+    begins (None: right after the query latent)."""
+    kv_off = q_rank if kv_off is None else int(kv_off)
+    assert proj.is_contiguous() and proj.shape[1] >= kv_off + kr + rot and pool.dtype == proj.dtype
+    assert q_rank == 0 or (cq.shape == (proj.shape[0], q_rank) and cq.is_contiguous() and cq.dtype == proj.dtype)
     stride, offset = _latent_pool(pool, layer, kr, rot, page_size)
-    _check(lib().st_latent_prepare(_p(proj), proj.shape[1], q_rank, _p(q_norm), _p(kv_norm), _f(eps), _p(inv_freq),
-                                   rot_dims, _p(cq), _p(pool), stride, offset, _p(positions), _p(seq_of_token),
+    _check(lib().st_latent_prepare(_p(proj), proj.shape[1], q_rank, kv_off, _p(q_norm), _p(kv_norm), _f(eps), _p(inv_freq),
+                                   rot_dims, int(neighbours), _f(rot_amp), _p(cq), _p(pool), stride, offset,
+                                   _p(positions), _p(seq_of_token),
                                    _p(slots), _p(block_table), block_table.shape[1], proj.shape[0], kr, rot, page_size,
                                    int(write_kv), _p(status), _dt(proj), _stream()), "latent_prepare")
 
 
 def latent_q_rotate(q: torch.Tensor, q_lat: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor,
-                    rot_dims: int, nh: int, dim: int, rot: int, kr: int) -> None:
-    """q [tokens, nh * (dim + rot)] -> the last ``rot`` numbers of every head's row of q_lat [tokens, nh, kr + rot]:
-    the head's rotated query part, turned by position."""
-    assert q.is_contiguous() and q_lat.is_contiguous() and q.dtype == q_lat.dtype
+                    rot_dims: int, nh: int, dim: int, rot: int, kr: int, neighbours: bool = False,
+                    rot_amp: float = 1.0) -> None:
+    """q [tokens, nh * (dim + rot)] (any row stride) -> the last ``rot`` numbers of every head's row of q_lat [tokens,
+    nh, kr + rot]: the head's rotated query part, turned by position (see ``latent_prepare``)."""
+    assert q.stride(1) == 1 and q_lat.is_contiguous() and q.dtype == q_lat.dtype
     assert q.shape[1] == nh * (dim + rot) and q_lat.shape == (q.shape[0], nh * (kr + rot))
-    _check(lib().st_latent_q_rotate(_p(q), _p(q_lat), _p(positions), _p(inv_freq), rot_dims, q.shape[0], nh, dim, rot,
+    _check(lib().st_latent_q_rotate(_p(q), q.stride(0), _p(q_lat), _p(positions), _p(inv_freq), rot_dims, int(neighbours),
+                                    _f(rot_amp), q.shape[0], nh, dim, rot,
                                     kr, _dt(q), _stream()), "latent_q_rotate")
 
 
@@ -896,8 +1023,9 @@ def latent_attention_plain(q_lat: torch.Tensor, pool: torch.Tensor, layer: int, 
                            block_table: torch.Tensor, nh: int, kr: int, rot: int, page_size: int, scale: float,
                            sink: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None,
                            status: Optional[torch.Tensor] = None, items: Optional[torch.Tensor] = None,
-                           n_items: int = 0) -> torch.Tensor:
-    """Causal attention in the latent space, one block per (token, head), float arithmetic for either type:
+                           n_items: int = 0, window: int = 0) -> torch.Tensor:
+    """Causal attention in the latent space, one block per (token, head), float arithmetic for either type (with a
+    ``window``: over the last ``window`` keys, the token's own among them):
     out [tokens, nh * kr] = gate * softmax-with-sink(scale * q_lat . [c | k_rot]) c.  ``gates``: a view
     [tokens, nh] (any row stride) of the heads' gate logits; ``sink`` float [nh]."""
     assert q_lat.is_contiguous() and out.is_contiguous() and out.shape == (q_lat.shape[0], nh * kr)
@@ -908,7 +1036,7 @@ def latent_attention_plain(q_lat: torch.Tensor, pool: torch.Tensor, layer: int, 
                                            _p(seq_of_token), _p(slots), _p(block_table), block_table.shape[1],
                                            n_items if items is not None else q_lat.shape[0], nh, kr, rot, page_size,
                                            _p(sink), _p(gates), gates.stride(0) if gates is not None else 0,
-                                           _f(scale), _p(status), _dt(q_lat), _stream()), "latent_attention_plain")
+                                           _f(scale), _p(status), _dt(q_lat), _stream(), window), "latent_attention_plain")
     return out
 
 
@@ -923,7 +1051,8 @@ def latent_attention(q_lat: torch.Tensor, pool: torch.Tensor, layer: int, out: t
                      rot: int, page_size: int, scale: float, sink: Optional[torch.Tensor] = None,
                      gates: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None, kernel: str = "auto",
                      q_start: Optional[torch.Tensor] = None, start_pos: Optional[torch.Tensor] = None, n_seqs: int = 0,
-                     lens=None, start=None, scratch=None, n_splits: Optional[int] = None) -> torch.Tensor:
+                     lens=None, start=None, scratch=None, n_splits: Optional[int] = None,
+                     window: int = 0) -> torch.Tensor:
     """Latent attention of the step's queries (see ``latent_attention_plain`` for the arguments).  kernel: "mma" = the
     tensor-core kernel over tiles of 64 (token, head) rows (bfloat16; it needs the step's requests: ``q_start``
     [n_seqs + 1], ``start_pos`` [n_seqs] on the device, or ``lens`` / ``start`` as host arrays), "plain" = the float
@@ -935,7 +1064,7 @@ def latent_attention(q_lat: torch.Tensor, pool: torch.Tensor, layer: int, out: t
         kernel = "mma" if latent_attention_mma_applies(q_lat, kr, rot) else "plain"
     if kernel == "plain":
         return latent_attention_plain(q_lat, pool, layer, out, positions, seq_of_token, slots, block_table, nh, kr, rot,
-                                      page_size, scale, sink, gates, status)
+                                      page_size, scale, sink, gates, status, window=window)
     if kernel != "mma":
         raise KernelError(f"latent_attention: no kernel named {kernel!r}")
     if not latent_attention_mma_applies(q_lat, kr, rot):
@@ -952,7 +1081,7 @@ def latent_attention(q_lat: torch.Tensor, pool: torch.Tensor, layer: int, out: t
         assert gates.dtype == q_lat.dtype and gates.stride(1) == 1 and gates.shape == (q_lat.shape[0], nh)
     n = q_lat.shape[0]
     if n_splits is None:
-        n_splits = int(lib().st_latent_attention_mma_splits(n, n_seqs, nh))
+        n_splits = int(lib().st_latent_attention_mma_splits(n, n_seqs, nh, window))
     partial = None
     if n_splits > 1:
         need = int(lib().st_latent_attention_mma_scratch(n, n_seqs, nh, kr, n_splits))
@@ -962,7 +1091,7 @@ def latent_attention(q_lat: torch.Tensor, pool: torch.Tensor, layer: int, out: t
                                          _p(start_pos), _p(slots), _p(block_table), block_table.shape[1],
                                          n, n_seqs, nh, kr, rot, page_size, _p(sink), _p(gates),
                                          gates.stride(0) if gates is not None else 0, _f(scale), n_splits, _p(partial),
-                                         _p(status), _stream()),
+                                         _p(status), _stream(), window),
            "latent_attention_mma")
     return out
 
@@ -994,11 +1123,34 @@ def _grouped_mma(a: torch.Tensor, k_dim: int, lda: int, a_goff: int, w_gstride: 
                                                        ctypes.c_longlong(w_gstride))))
 
 
+def _route_rule(scores: str, groups, renorm: bool, scale: float):
+    if scores not in ("softmax", "sigmoid"):
+        raise KernelError(f"router scores are 'softmax' or 'sigmoid', not {scores!r}")
+    count, keep = groups if groups else (0, 0)
+    return int(scores == "sigmoid"), int(count), int(keep), int(renorm), _f(scale)
+
+
+def moe_choose(logits: torch.Tensor, n_experts: int, top: int, positions: Optional[torch.Tensor] = None,
+               renorm: bool = False, scores: str = "softmax", groups: Optional[Sequence[int]] = None, scale: float = 1.0):
+    """The choice of ``moe_route`` alone, from float32 router logits [tokens, >= n_experts] that a product left."""
+    n = logits.shape[0]
+    assert logits.dtype == torch.float32 and logits.is_contiguous() and logits.shape[1] >= n_experts
+    experts = torch.empty((n, top), dtype=torch.int32, device=logits.device)
+    weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    _check(lib().st_moe_choose(_p(logits), logits.shape[1], n, n_experts, top, *_route_rule(scores, groups, renorm, scale),
+                               _p(positions), _p(experts), _p(weights), _stream()), "moe_choose")
+    return experts, weights
+
+
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, positions: Optional[torch.Tensor] = None,
-              w_gate: Optional[torch.Tensor] = None, renorm: bool = False):
+              w_gate: Optional[torch.Tensor] = None, renorm: bool = False, scores: str = "softmax",
+              groups: Optional[Sequence[int]] = None, scale: float = 1.0):
     """-> (experts int32 [tokens, top], weights float [tokens, top], gate float [tokens] or None).  Router logits,
     softmax over all experts and the choice in float; ``w_router`` float [experts, width]; ``w_gate`` float [width]:
-    also sigmoid(w_gate . h) per token.  Tokens at a negative position get expert -1."""
+    also sigmoid(w_gate . h) per token.  Tokens at a negative position get expert -1.  ``scores`` "sigmoid": the scores
+    are sigmoids of the logits.  ``groups`` (count, keep): the experts form ``count`` equal groups of neighbours, only the
+    ``keep`` with the largest sums of their two largest scores can be chosen from.  The weights (divided by their sum
+    with ``renorm``) are multiplied by ``scale``."""
     n, width = h.shape
     assert h.is_contiguous() and w_router.dtype == torch.float32 and w_router.is_contiguous() and w_router.shape[1] == width
     experts = torch.empty((n, top), dtype=torch.int32, device=h.device)
@@ -1006,7 +1158,8 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, positions: Opti
     gate = torch.empty((n,), dtype=torch.float32, device=h.device) if w_gate is not None else None
     if w_gate is not None:
         assert w_gate.dtype == torch.float32 and w_gate.numel() == width and w_gate.is_contiguous()
-    _check(lib().st_moe_route(_p(h), n, width, _p(w_router), w_router.shape[0], top, int(renorm), _p(w_gate),
+    _check(lib().st_moe_route(_p(h), n, width, _p(w_router), w_router.shape[0], top,
+                              *_route_rule(scores, groups, renorm, scale), _p(w_gate),
                               _p(positions), _p(experts), _p(weights), _p(gate), _dt(h), _stream()), "moe_route")
     return experts, weights, gate
 
@@ -1040,7 +1193,7 @@ def gemm_experts(a: torch.Tensor, w: torch.Tensor, order: ExpertOrder, gather: b
                  act: str = "none") -> torch.Tensor:
     """One product per expert over the rows the order gives it: out [items, n_out] in sorted order.
     ``gather``: the rows of ``a`` are the tokens (row of item i = i // top), else ``a`` is already in sorted order.
-    w [experts, n_out (twice with ``gated``: gate rows, then up rows), k]; gated: out = act(gate) * up."""
+    w [experts, n_out (twice with ``gated``: gate rows, then up rows), k]; out = act(product), gated: act(gate) * up."""
     assert a.is_contiguous() and w.is_contiguous() and w.dim() == 3 and a.dtype == w.dtype and a.shape[1] == w.shape[2]
     n_out = w.shape[1] // 2 if gated else w.shape[1]
     out = torch.empty((order.n_items, n_out), dtype=a.dtype, device=a.device)
@@ -1127,10 +1280,11 @@ def gqa_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias: Op
                 q_out: torch.Tensor, pool: torch.Tensor, layer: int, positions: torch.Tensor,
                 seq_of_token: torch.Tensor, slots: torch.Tensor, block_table: torch.Tensor, nh: int, nkv: int,
                 dim: int, vd: int, page_size: int, status: Optional[torch.Tensor], write_kv: bool = True,
-                norm_eps: float = 0.0) -> None:
+                norm_eps: float = 0.0, neighbours: bool = False, rot_amp: float = 1.0) -> None:
     """Queries, keys and values of a step from the fused projection ``proj`` [tokens, columns] (queries at column
     q_off, keys at k_off, values at v_off): plus ``bias`` (float32, one number per column of proj, or None); the
-    first ``rot_dims`` dimensions of every query and key head rotated by position in the halves layout; queries
+    first ``rot_dims`` dimensions of every query and key head rotated by position in the halves layout (or in pairs of
+    ``neighbours``; sine and cosine times ``rot_amp``); queries
     times 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1); queries to ``q_out`` [tokens, nh * dim], keys and
     values into their pages (``write_kv`` False: queries only).  ``norm_eps`` > 0: after the rotation every query and
     key head is divided by its root mean square over ``dim`` (eps inside the root, no weight)."""
@@ -1143,7 +1297,7 @@ def gqa_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias: Op
                                 _f(temp_coef), temp_every, _p(q_out), _p(pool), stride, off, _p(positions),
                                 _p(seq_of_token), _p(slots), _p(block_table), block_table.shape[1], proj.shape[0], nh,
                                 nkv, dim, vd, page_size, int(write_kv), _p(status), _dt(proj), _stream(),
-                                _f(norm_eps)), "gqa_prepare")
+                                _f(norm_eps), int(neighbours), _f(rot_amp)), "gqa_prepare")
 
 
 def _sink_args(sink, nh: int):
@@ -1170,12 +1324,12 @@ def gqa_attention_plain(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                         dim: int, vd: int, page_size: int, scale: float, window: int, keep_first: int,
                         sink: Optional[float], gate: Optional[torch.Tensor], gate_off: int, out_scale: float,
                         status: Optional[torch.Tensor] = None, items: Optional[torch.Tensor] = None,
-                        n_items: Optional[int] = None) -> torch.Tensor:
+                        n_items: Optional[int] = None, gate_heads: bool = False) -> torch.Tensor:
     """Grouped attention of every token of the step (or of those ``items`` lists) over the paged cache, in float
     arithmetic for either storage type.  ``window`` 0: all keys up to the query; else the last ``window`` keys and
     the request's first ``keep_first``.  ``sink``: a logit that joins the softmax's denominator (None: none).
     ``gate`` [tokens, columns]: the head's result is multiplied by sigmoid of its columns from ``gate_off`` on.
-    ``sink`` may also be a float32 tensor [heads]: a logit per head."""
+    ``sink`` may also be a float32 tensor [heads]: a logit per head.  ``gate_heads``: one gate column per head."""
     assert q.is_contiguous() and out.is_contiguous() and out.shape == (q.shape[0], nh * vd)
     stride, off, gate_ptr, gate_ld = _gqa_tail(pool, layer, nkv, dim, vd, page_size, scale, window, keep_first, sink,
                                                gate, gate_off, out_scale)
@@ -1185,7 +1339,7 @@ def gqa_attention_plain(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                                         _p(seq_of_token), _p(slots), _p(block_table), block_table.shape[1], n, nh, nkv,
                                         dim, vd, page_size, _f(scale), window, keep_first, has_sink,
                                         sink_one, gate_ptr, gate_ld, _f(out_scale), _p(status), _dt(q),
-                                        _stream(), sinks), "gqa_attention_plain")
+                                        _stream(), sinks, int(gate_heads)), "gqa_attention_plain")
     return out
 
 
@@ -1260,7 +1414,7 @@ def gqa_attention_tiles(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                         slots: torch.Tensor, block_table: torch.Tensor, nh: int, nkv: int, dim: int, vd: int,
                         page_size: int, scale: float, window: int, keep_first: int, sink: Optional[float],
                         gate: Optional[torch.Tensor], gate_off: int, out_scale: float,
-                        status: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        status: Optional[torch.Tensor] = None, gate_heads: bool = False) -> torch.Tensor:
     """The same attention for tiles of ``tile_rows`` query rows (tiles: int32 [n_tiles, 2] = request of the step,
     offset of the tile among its new tokens) on the warp-level tensor cores, bfloat16 only."""
     if not (q.dtype == torch.bfloat16 and bool(lib().st_gqa_attention_tiles_applies(dim, vd))):
@@ -1273,7 +1427,7 @@ def gqa_attention_tiles(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                                         _p(q_start), _p(start_pos), _p(slots), _p(block_table), block_table.shape[1],
                                         nh, nkv, dim, vd, page_size, _f(scale), window, keep_first,
                                         has_sink, sink_one, gate_ptr, gate_ld, _f(out_scale),
-                                        _p(status), _stream(), sinks), "gqa_attention_tiles")
+                                        _p(status), _stream(), sinks, int(gate_heads)), "gqa_attention_tiles")
     return out
 
 
@@ -1282,7 +1436,7 @@ def gqa_attention_single(q: torch.Tensor, pool: torch.Tensor, layer: int, out: t
                          dim: int, vd: int, page_size: int, scale: float, window: int, keep_first: int,
                          sink: Optional[float], gate: Optional[torch.Tensor], gate_off: int, out_scale: float,
                          status: Optional[torch.Tensor] = None, items: Optional[torch.Tensor] = None,
-                         n_items: Optional[int] = None) -> torch.Tensor:
+                         n_items: Optional[int] = None, gate_heads: bool = False) -> torch.Tensor:
     """The same attention token by token in bfloat16, one block per (token, key/value head) for all the query heads
     that read it; ``items`` as for the plain kernel."""
     if not (q.dtype == torch.bfloat16 and bool(lib().st_gqa_attention_single_applies(nh, nkv, dim, vd))):
@@ -1296,8 +1450,8 @@ def gqa_attention_single(q: torch.Tensor, pool: torch.Tensor, layer: int, out: t
     _check(lib().st_gqa_attention_single(_p(q), _p(pool), stride, off, _p(out), _p(items), _p(positions),
                                          _p(seq_of_token), _p(slots), _p(block_table), block_table.shape[1], n, nh, nkv,
                                          dim, vd, page_size, _f(scale), window, keep_first, has_sink,
-                                         sink_one, gate_ptr, gate_ld, _f(out_scale), _p(status), _stream(), sinks),
-           "gqa_attention_single")
+                                         sink_one, gate_ptr, gate_ld, _f(out_scale), _p(status), _stream(), sinks,
+                                         int(gate_heads)), "gqa_attention_single")
     return out
 
 

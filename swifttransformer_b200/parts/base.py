@@ -48,6 +48,8 @@ class Delta:
     value: Optional[torch.Tensor]        # [N, width], activation dtype, or None
     bias: Optional[torch.Tensor] = None  # [width] float32
     parts: Optional[torch.Tensor] = None  # [n, N, width] float32
+    # what the sub-layer's first product gave for the rows its block handed it (see ``RowTaker``): a view [N, rows]
+    extra: Optional[torch.Tensor] = None
 
 
 @dataclasses.dataclass(frozen=True)
@@ -137,6 +139,32 @@ class StepPlan:
         """What the mixers get from ``ctx.plan(name)``: built over ``dev`` (the device copy of the words)
         for a step described by ``key`` (an exact key, or a padded one when the step is recorded)."""
         return None
+
+
+def stack_rows(mats: List[torch.Tensor], multiple: int = 8) -> Tuple[torch.Tensor, List[int]]:
+    """Matrices [out, in] of one input stacked into one, each filled up with zero rows to a multiple of ``multiple`` (so
+    that every member's columns of the product begin on an aligned address); -> (matrix, first row of each member)."""
+    out, offsets, at = [], [], 0
+    for m in mats:
+        offsets.append(at)
+        fill = -m.shape[0] % multiple
+        out.append(m)
+        if fill:
+            out.append(m.new_zeros((fill, m.shape[1])))
+        at += m.shape[0] + fill
+    return torch.cat(out, dim=0).contiguous(), offsets
+
+
+class RowTaker:
+    """A sub-layer whose first product can carry rows of its block: a block that needs a product of the sub-layer's own
+    input (the logits of a gate on its result) hands the matrix over before ``bind`` and finds the columns in
+    ``Delta.extra``, so that both are one product.  A sub-layer without ``take_rows`` leaves the product to the block."""
+
+    extra_rows: Optional[torch.Tensor] = None
+
+    def take_rows(self, w: torch.Tensor) -> bool:
+        self.extra_rows = w
+        return True
 
 
 class Mixer(Part):

@@ -14,6 +14,9 @@ reentry   (no sub-layers; opens a pass over a stretch of layers that runs severa
 hyper_pre_norm (n copies x_1..x_n of the residual rows instead of one; sub-layer f with coefficients a, b, M):
     u = sum_s a_s x_s;  y = f(c(norm(u)));  x_t' = sum_s M[s, t] x_s + b_t y        c: an optional short
     convolution over time, c(h) = h + conv(h); the model's residual rows are the sum of the copies
+gated_sandwich (a norm before and after each sub-layer, and a gate on its result from the sub-layer's own input):
+    h = norm(x);  x' = x + norm_b(sigmoid(R h + r) * f(h))      f: the mixer, then the feed-forward; and after both an
+    optional side input looked up by token: x' = x + norm_s(P (gelu_tanh(K x) * e_token))
 
 The residual stream is float32 for every storage type.  A block leaves the
 feed-forward's result as ``pending``: the next norm kernel (of the next block
@@ -42,6 +45,18 @@ class ResidualStream:
     lanes: Optional[torch.Tensor] = None   # [n, N, width] float32: the copies of a model with several residual streams
     # (mix [n, n], out [n], y [N, width]): the update of the copies that the last sub-layer left to the next reader
     lanes_pending: Optional[tuple] = None
+    # (y [N, width], gate logits or None, gate bias or None, gain [width], eps): x is still to be given
+    # gain * rms_unit(y * sigmoid(gate + bias)) by the next reader
+    normed_pending: Optional[tuple] = None
+
+    def settle_normed(self, ctx: Any = None, norm: Optional[Norm] = None, out_act: Optional[torch.Tensor] = None) -> None:
+        """Add the normed result that the last sub-layer left pending to x; in the same pass, with ``out_act``, what
+        reads x next: norm(x), or x itself without a norm, in the activation type."""
+        y, gate, bias, gain, eps = self.normed_pending
+        self.normed_pending, self.act = None, None
+        ops.gated_norm_add(self.x, y, gate, bias, gain, eps, ctx.positions if ctx is not None else None,
+                           next_gain=norm.gamma if norm is not None else None, next_eps=norm.eps if norm is not None else 0.0,
+                           out_act=out_act)
 
     def settle_lanes(self) -> None:
         """Apply the update of the copies that the last sub-layer left pending."""
@@ -51,8 +66,11 @@ class ResidualStream:
             self.lanes_pending = None
 
     def fold(self) -> None:
-        """A model with several residual streams: x <- their sum (what the final norm and the tools that look at
-        the residual rows read); the copies themselves stay as they are."""
+        """Bring x up to date with what the last sub-layer left to its reader.  A model with several residual streams:
+        x <- their sum (what the final norm and the tools that look at the residual rows read); the copies themselves
+        stay as they are."""
+        if self.normed_pending is not None:
+            self.settle_normed()
         if self.lanes is not None:
             self.settle_lanes()
             ops.hc_sum(self.lanes, out=self.x)
@@ -60,6 +78,8 @@ class ResidualStream:
 
     def materialise(self, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """x + pending in the activation dtype (all rows, folding pending into x; or only ``rows``)."""
+        if self.normed_pending is not None:
+            self.settle_normed()
         if rows is None and self.pending is None and self.act is not None:
             return self.act
         n = rows.numel() if rows is not None else self.x.shape[0]
@@ -357,4 +377,95 @@ class HyperPreNormBlock(Block):
             h = self._input(1, stream, self.norm2, ctx, tail2)
             y = self._rows(self.feed_forward.forward(h, ctx), stream)
             stream.lanes_pending = (self.coef[1][1], self.coef[1][2], y)
+        stream.pending, stream.act = None, None
+
+
+@BLOCKS.register("gated_sandwich")
+class GatedSandwichBlock(Block):
+    """For the mixer and then the feed-forward (which may be absent): h = norm(x); x <- x + norm_b(sigmoid(R h + r) * f(h)).
+    ``gate_names``: the tensors of (R [width, width], its bias being the name + ``.b``) for the two sub-layers; ``norm1b``
+    and ``norm2b`` the norms of the sub-layers' results.  Then, with ``side`` (a TokenSide) and ``side_names`` {"gate"
+    [dim, width], "proj" [width, dim], "norm" [width]}, the layer's own input by token:
+    x <- x + norm_s(P (gelu_tanh(K x) * e)), e the part ``layer`` of the token's row.
+
+    R rides in the sub-layer's first product where that can carry it (RowTaker), else it is a product of its own.  Gate,
+    norm of the result, residual sum and the norm (or the copy) that the next reader of x needs are one kernel: a
+    sub-layer leaves its result and gate logits pending (``ResidualStream.normed_pending``) to that reader."""
+
+    def __init__(self, mixer: Mixer, feed_forward: Optional[FeedForward], norm1: Norm, norm1b: Norm, width: int,
+                 gate_names: tuple, norm2: Optional[Norm] = None, norm2b: Optional[Norm] = None, side: Any = None,
+                 side_names: Optional[dict] = None, layer: int = 0, eps: float = 1e-6, bias_suffix: str = ".b"):
+        if (feed_forward is None) != (norm2 is None) or (feed_forward is None) != (norm2b is None):
+            raise ValueError("a block has norms around a feed-forward exactly when it has one")
+        if (side is None) != (side_names is None):
+            raise ValueError("a side input needs its table and its tensors' names")
+        super().__init__(mixer, feed_forward, norm1, norm2)
+        self.norm1b, self.norm2b, self.width, self.eps = norm1b, norm2b, int(width), float(eps)
+        self.gate_names, self.suffix = tuple(gate_names), bias_suffix
+        self.side, self.side_names, self.layer = side, dict(side_names) if side_names else None, int(layer)
+        self.n_sub = 1 if feed_forward is None else 2
+        self.gate_w, self.gate_b = [None, None], [None, None]
+        self.w_side_gate = self.w_side_proj = self.side_gain = None
+
+    def children(self) -> List[Part]:
+        parts = (self.norm1, self.mixer, self.norm1b, self.norm2, self.feed_forward, self.norm2b)
+        return [p for p in parts if p is not None]
+
+    def param_specs(self):
+        from ..weights.spec import GAIN, MATRIX, VECTOR, ParamSpec
+        W, specs = self.width, []
+        for name in self.gate_names[:self.n_sub]:
+            specs += [ParamSpec(name, (W, W), MATRIX), ParamSpec(name + self.suffix, (W,), VECTOR)]
+        if self.side is not None:
+            n, dim = self.side_names, self.side.dim
+            specs += [ParamSpec(n["gate"], (dim, W), MATRIX), ParamSpec(n["proj"], (W, dim), MATRIX),
+                      ParamSpec(n["norm"], (W,), GAIN)]
+        return specs
+
+    def bind(self, tensors) -> None:
+        # (a block is bound before its children: the sub-layers find the rows when they stack their own)
+        for i, sub in enumerate((self.mixer, self.feed_forward)[:self.n_sub]):
+            w, self.gate_b[i] = tensors.pop(self.gate_names[i]), tensors[self.gate_names[i] + self.suffix]
+            if not (hasattr(sub, "take_rows") and sub.take_rows(w)):
+                self.gate_w[i] = w
+        if self.side is not None:
+            n = self.side_names
+            self.w_side_gate, self.w_side_proj = tensors[n["gate"]], tensors[n["proj"]]
+            self.side_gain = tensors[n["norm"]]
+
+    def param_bytes(self) -> int:
+        mats = [w for w in self.gate_w + [self.w_side_gate, self.w_side_proj] if w is not None]
+        return sum(w.numel() * w.element_size() for w in mats)
+
+    def _read(self, stream: ResidualStream, norm: Norm, ctx: Any) -> torch.Tensor:
+        if stream.normed_pending is None:
+            h = norm.apply(stream.x, stream.pending, act_dtype=stream.act_dtype)
+            stream.pending = None
+            return h
+        h = torch.empty(stream.x.shape, dtype=stream.act_dtype, device=stream.x.device)
+        stream.settle_normed(ctx, norm, h)
+        return h
+
+    def _leave(self, stream: ResidualStream, i: int, h: torch.Tensor, delta: Delta, norm: Norm) -> None:
+        assert delta.bias is None and delta.parts is None
+        gate = delta.extra if self.gate_w[i] is None else ops.linear(h, self.gate_w[i])
+        stream.normed_pending = (delta.value, gate, self.gate_b[i], norm.gamma, norm.eps)
+
+    def forward(self, stream: ResidualStream, ctx: Any, cache: Any) -> None:
+        h = self._read(stream, self.norm1, ctx)
+        self._leave(stream, 0, h, self.mixer.forward(h, ctx, cache), self.norm1b)
+        if self.feed_forward is not None:
+            h = self._read(stream, self.norm2, ctx)
+            self._leave(stream, 1, h, self.feed_forward.forward(h, ctx), self.norm2b)
+        if self.side is not None:
+            if stream.act_dtype == torch.float32:
+                stream.settle_normed(ctx)
+                a = stream.x
+            else:
+                a = torch.empty(stream.x.shape, dtype=stream.act_dtype, device=stream.x.device)
+                stream.settle_normed(ctx, None, a)
+            s = ops.linear(a, self.w_side_gate, out_dtype=torch.float32)
+            g = ops.side_input(s, self.side.table, self.layer * self.side.dim, ctx.token_ids)
+            y = ops.linear(g, self.w_side_proj, out_dtype=torch.float32)
+            stream.normed_pending = (y, None, None, self.side_gain, self.eps)
         stream.pending, stream.act = None, None

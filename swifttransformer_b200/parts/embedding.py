@@ -66,6 +66,21 @@ class Embedding(Part):
         return self.project_in.numel() * self.project_in.element_size() if self.project_in is not None else 0
 
 
+class TokenSide(Part):
+    """A second table looked up by token that every layer reads a part of: row [layers * dim], layer i's part the columns
+    i * dim .. (i + 1) * dim - 1.  Blocks with a side input hold a reference to it."""
+
+    def __init__(self, vocab: int, layers: int, dim: int, name: str):
+        self.vocab, self.layers, self.dim, self.name = vocab, layers, dim, name
+        self.table: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> List[ParamSpec]:
+        return [ParamSpec(self.name, (self.vocab, self.layers * self.dim), TABLE)]
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.table = tensors[self.name]
+
+
 class OutputHead(Part):
     """logits = (project_out . h) . table^T as float32; with ``scale`` and ``softcap`` (0: none),
     logits <- softcap * tanh(logits * scale / softcap)."""

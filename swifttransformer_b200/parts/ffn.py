@@ -13,28 +13,31 @@ import torch
 
 from .. import ops
 from ..weights.spec import MATRIX, VECTOR, ParamSpec
-from .base import FEED_FORWARDS, Delta, FeedForward
+from .base import FEED_FORWARDS, Delta, FeedForward, RowTaker, stack_rows
 
 
 @FEED_FORWARDS.register("dense")
 class DenseFFN(FeedForward):
-    def __init__(self, hidden: int, inner: int, activation: str, fc1_name: str, fc2_name: str, bias: bool = True):
+    """The matrices are the tensors ``fc1_name`` / ``fc2_name`` + ``weight_suffix``."""
+
+    def __init__(self, hidden: int, inner: int, activation: str, fc1_name: str, fc2_name: str, bias: bool = True,
+                 weight_suffix: str = ".weight"):
         if activation not in ops.ACT_CODES:
             raise ValueError(f"activation '{activation}' is not supported ({', '.join(ops.ACT_CODES)})")
         self.hidden, self.inner, self.activation, self.bias = hidden, inner, activation, bias
-        self.fc1_name, self.fc2_name = fc1_name, fc2_name
+        self.fc1_name, self.fc2_name, self.suffix = fc1_name, fc2_name, weight_suffix
         self.w1 = self.b1 = self.w2 = self.b2 = self.b1_bf16 = None
 
     def param_specs(self) -> List[ParamSpec]:
-        specs = [ParamSpec(self.fc1_name + ".weight", (self.inner, self.hidden), MATRIX),
-                 ParamSpec(self.fc2_name + ".weight", (self.hidden, self.inner), MATRIX)]
+        specs = [ParamSpec(self.fc1_name + self.suffix, (self.inner, self.hidden), MATRIX),
+                 ParamSpec(self.fc2_name + self.suffix, (self.hidden, self.inner), MATRIX)]
         if self.bias:
             specs += [ParamSpec(self.fc1_name + ".bias", (self.inner,), VECTOR),
                       ParamSpec(self.fc2_name + ".bias", (self.hidden,), VECTOR)]
         return specs
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
-        self.w1, self.w2 = tensors[self.fc1_name + ".weight"], tensors[self.fc2_name + ".weight"]
+        self.w1, self.w2 = tensors[self.fc1_name + self.suffix], tensors[self.fc2_name + self.suffix]
         if self.bias:
             self.b1, self.b2 = tensors[self.fc1_name + ".bias"], tensors[self.fc2_name + ".bias"]
             if self.w1.dtype == torch.bfloat16:
@@ -69,7 +72,7 @@ class DenseFFN(FeedForward):
 
 
 @FEED_FORWARDS.register("gated")
-class GatedFFN(FeedForward):
+class GatedFFN(RowTaker, FeedForward):
     """z = down(act(gate h) * (up h)), no biases.  The gate and up matrices are stacked at load time so that one
     product gives both; ``activation`` is any of ops.ACT_CODES (the tanh form of GELU, SiLU, ...).  ``float_out``:
     the down product leaves its float sums as they are (a block that adds two sub-layers' results takes them so)."""
@@ -82,6 +85,7 @@ class GatedFFN(FeedForward):
         self.hidden, self.inner, self.activation = hidden, inner, activation
         self.gate_name, self.up_name, self.down_name = gate_name, up_name, down_name
         self.w_gu = self.w_down = None
+        self.extra_off = self.extra_n = 0
 
     def param_specs(self) -> List[ParamSpec]:
         return [ParamSpec(self.gate_name, (self.inner, self.hidden), MATRIX),
@@ -90,11 +94,16 @@ class GatedFFN(FeedForward):
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.w_gu = torch.cat([tensors.pop(self.gate_name), tensors.pop(self.up_name)], dim=0).contiguous()
+        if self.extra_rows is not None:
+            self.w_gu, (_, self.extra_off) = stack_rows([self.w_gu, self.extra_rows])
+            self.extra_n, self.extra_rows = self.extra_rows.shape[0], None
         self.w_down = tensors[self.down_name]
 
     def forward(self, h: torch.Tensor, ctx: Any) -> Delta:
-        u = ops.gated_act(ops.linear(h, self.w_gu), self.activation)
-        return Delta(ops.linear(u, self.w_down, out_dtype=torch.float32 if self.float_out else None))
+        gu = ops.linear(h, self.w_gu)
+        u = ops.gated_act(gu, self.activation, self.inner)
+        extra = gu[:, self.extra_off:self.extra_off + self.extra_n] if self.extra_n else None
+        return Delta(ops.linear(u, self.w_down, out_dtype=torch.float32 if self.float_out else None), extra=extra)
 
     def param_bytes(self) -> int:
         return (self.w_gu.numel() + self.w_down.numel()) * self.w_gu.element_size()

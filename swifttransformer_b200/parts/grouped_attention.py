@@ -3,7 +3,7 @@
 Per query head a (key/value head a // (heads / kv_heads)), key/query size ``dim``, value size ``vdim``:
 
     q, k, v   = the projections of the mixer's input (+ biases)
-    q, k      <- rotated by position on the first ``rot.dims`` dimensions (a ``rotary_halves`` encoding), or not
+    q, k      <- rotated by position on the first ``rot.dims`` dimensions (a rotary encoding: halves or pairs), or not
     q         <- q * (1 + coef * ln(floor((p + 1) / every) + 1))            (``q_temp`` = (coef, every), or None)
     s_j       = scale * q . k_j  over the keys the query at p sees: j <= p, and with a ``window``
                 p - j < window or j < keep_first
@@ -35,11 +35,11 @@ import torch
 from .. import ops
 from ..weights.spec import MATRIX, VECTOR, ParamSpec
 from .attention import PagedAttentionPlan
-from .base import MIXERS, Delta, Mixer, PagedKVSpec, StepPlan
+from .base import MIXERS, Delta, Mixer, PagedKVSpec, RowTaker, StepPlan, stack_rows
 
 
 @MIXERS.register("grouped_attention")
-class GroupedAttention(Mixer):
+class GroupedAttention(RowTaker, Mixer):
     """names: tensor names of the projections {"q","k","v","o"} and, with ``gate``, "g" ([out, in] matrices);
     a projection's bias is its name + ``bias_suffix``.  ``qkv_bias`` / ``o_bias``: which projections have one."""
 
@@ -79,6 +79,7 @@ class GroupedAttention(Mixer):
         self.gw = (num_heads if self.gate_heads else num_heads * vdim) if gate else 0
         self.w_in = self.b_in = self.w_o = self.b_o = self.sinks = self.talk = None
         self._plan: Optional[PagedAttentionPlan] = None
+        self.extra_off = self.extra_n = 0
 
     # ------------------------------------------------------------ tensors
     def _projections(self):
@@ -115,6 +116,10 @@ class GroupedAttention(Mixer):
             else:
                 biases.append(torch.zeros(rows, dtype=torch.float32, device=w.device))
         self.w_in = torch.cat(mats, dim=0).contiguous()
+        if self.extra_rows is not None:
+            self.w_in, (_, self.extra_off) = stack_rows([self.w_in, self.extra_rows])
+            self.extra_n, self.extra_rows = self.extra_rows.shape[0], None
+            biases.append(torch.zeros(self.w_in.shape[0] - sum(b.numel() for b in biases), device=self.w_in.device))
         self.b_in = torch.cat(biases, dim=0).contiguous() if self.qkv_bias else None
         self.w_o = tensors.pop(n["o"])
         self.b_o = tensors.pop(n["o"] + self.suffix) if self.o_bias else None
@@ -148,11 +153,13 @@ class GroupedAttention(Mixer):
         ops.gqa_prepare(proj, 0, self.qw, self.qw + self.kw, self.b_in, rot.inv_freq(h.device) if rot_dims else None,
                         rot_dims, temp[0], temp[1], q, cache.pool, cache.layer, ctx.positions, ctx.seq_of_token,
                         ctx.slots, cache.block_table, self.nh, self.nkv, self.dim, self.vdim, ps, ctx.status,
-                        write_kv=self.own_kv and cache.writable, norm_eps=self.qk_norm_eps)
+                        write_kv=self.own_kv and cache.writable, norm_eps=self.qk_norm_eps,
+                        neighbours=rot is not None and rot.neighbours, rot_amp=rot.amplitude if rot is not None else 1.0)
+        extra = proj[:, self.extra_off:self.extra_off + self.extra_n] if self.extra_n else None
         o = torch.empty((n, self.nh * self.vdim), dtype=h.dtype, device=h.device)
         gate, gate_off = (proj, self.qw + self.kw + self.vw) if self.gate else (None, 0)
         sink = self.sinks if self.sinks is not None else self.sink
-        if self.talk is not None or self.gate_heads:
+        if self.talk is not None:
             # every head's weights of a key meet before the values: the heads of a token are served together
             args = (cache.pool, cache.layer, o)
             tail = (self.nh, self.nkv, self.dim, self.vdim, ps, self.scale, self.window or 0, self.keep_first, self.talk,
@@ -178,7 +185,7 @@ class GroupedAttention(Mixer):
                     else:
                         ops.talk_attention_plain(q, *args, *rows, *tail, status=ctx.status, items=plan.items,
                                                  n_items=plan.n_items)
-            return Delta(ops.linear(o, self.w_o, out_dtype=torch.float32 if self.float_out else None), self.b_o)
+            return Delta(ops.linear(o, self.w_o, out_dtype=torch.float32 if self.float_out else None), self.b_o, extra=extra)
         consts = (self.nh, self.nkv, self.dim, self.vdim, ps, self.scale, self.window or 0, self.keep_first, sink,
                   gate, gate_off, self.out_scale)
         if ops.gqa_attention_fast_applies(q, self.nh, self.nkv, self.dim, self.vdim):
@@ -186,15 +193,15 @@ class GroupedAttention(Mixer):
             if plan.n_tiles:
                 ops.gqa_attention_tiles(q, cache.pool, cache.layer, o, plan.tiles, plan.n_tiles, self._plan.tile_rows,
                                         ctx.q_start, ctx.start_pos, ctx.slots, cache.block_table, *consts,
-                                        status=ctx.status)
+                                        status=ctx.status, gate_heads=self.gate_heads)
             if plan.n_items:
                 ops.gqa_attention_single(q, cache.pool, cache.layer, o, ctx.positions, ctx.seq_of_token, ctx.slots,
                                          cache.block_table, *consts, status=ctx.status, items=plan.items,
-                                         n_items=plan.n_items)
+                                         n_items=plan.n_items, gate_heads=self.gate_heads)
         else:
             ops.gqa_attention_plain(q, cache.pool, cache.layer, o, ctx.positions, ctx.seq_of_token, ctx.slots,
-                                    cache.block_table, *consts, status=ctx.status)
-        return Delta(ops.linear(o, self.w_o, out_dtype=torch.float32 if self.float_out else None), self.b_o)
+                                    cache.block_table, *consts, status=ctx.status, gate_heads=self.gate_heads)
+        return Delta(ops.linear(o, self.w_o, out_dtype=torch.float32 if self.float_out else None), self.b_o, extra=extra)
 
     def _sink_vector(self, device) -> Optional[torch.Tensor]:
         """The extra term's logit of every head for the kernels that take one per head (None: no extra term)."""

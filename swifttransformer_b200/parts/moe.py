@@ -1,4 +1,4 @@
-"""A routed mixture of gated feed-forward experts, with an optional shared expert.
+"""A routed mixture of feed-forward experts, gated or plain, with an optional shared expert.
 
     z = W_r h  (float)           s = softmax(z) over all experts
     the ``top`` experts with the largest s are chosen; their weights are their s (divided by their sum only with
@@ -6,7 +6,9 @@
     out = sum over the chosen e of s_e * down_e(act(gate_e h) * (up_e h))
           + sigmoid(w_sg . h) * down_s(act(gate_s h) * (up_s h))          the shared expert, for every token
 
-With ``limit`` the experts are clamped gated units instead: g = min(gate_e h, limit), u = clamp(up_e h, -limit, limit),
+``scores`` "sigmoid": s = sigmoid(z).  ``groups`` (count, keep): the experts form ``count`` equal groups of neighbours; the
+choice is among the ``keep`` groups with the largest sums of their two largest scores.  ``scale`` multiplies the weights.
+``gated`` False: the experts are down_e(act(up_e h)).  With ``limit`` the experts are clamped gated units instead: g = min(gate_e h, limit), u = clamp(up_e h, -limit, limit),
 down_e(g * sigmoid(alpha * g) * (u + shift)).
 
 On the device the step's (token, choice) items are grouped by expert (``ops.moe_sort``), two grouped products run
@@ -15,7 +17,7 @@ adds the gated shared expert, in float.  Nothing comes back to the host, so step
 """
 from __future__ import annotations
 
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Sequence
 
 import torch
 
@@ -24,16 +26,21 @@ from ..weights.spec import MATRIX, VECTOR, ParamSpec
 from .base import FEED_FORWARDS, Delta, FeedForward, Part
 
 
+# steps of more tokens take the router logits from a product (few tokens: product and choice are one kernel)
+ROUTE_PRODUCT_MIN_ROWS = 16
+
+
 @FEED_FORWARDS.register("routed_experts")
 class RoutedExperts(FeedForward):
-    """expert_names: per expert {"gate", "up", "down"} tensor names; router_name: [experts, hidden] (kept in float);
+    """expert_names: per expert {"gate", "up", "down"} tensor names (no "gate" with ``gated`` False); router_name: [experts, hidden] (kept in float);
     shared: a feed-forward part for every token or None, with shared_gate_name ([1, hidden] or [hidden], float) the
     weight of its sigmoid gate (None: the shared expert is added as it is)."""
 
     def __init__(self, hidden: int, inner: int, num_experts: int, top: int, activation: str,
                  expert_names: List[Dict[str, str]], router_name: str, shared: Optional[FeedForward] = None,
                  shared_gate_name: Optional[str] = None, renormalise: bool = False, limit: Optional[float] = None,
-                 alpha: float = 1.0, shift: float = 0.0):
+                 alpha: float = 1.0, shift: float = 0.0, scores: str = "softmax", groups: Optional[Sequence[int]] = None,
+                 scale: float = 1.0, gated: bool = True):
         self.limit, self.alpha, self.shift = (float(limit) if limit else None), float(alpha), float(shift)
         if activation not in ops.ACT_CODES:
             raise ValueError(f"activation '{activation}' is not supported ({', '.join(ops.ACT_CODES)})")
@@ -42,7 +49,15 @@ class RoutedExperts(FeedForward):
         self.hidden, self.inner, self.n_experts, self.top, self.activation = hidden, inner, num_experts, top, activation
         self.expert_names, self.router_name = expert_names, router_name
         self.shared, self.shared_gate_name, self.renormalise = shared, shared_gate_name, renormalise
-        self.w_router = self.w_gu = self.w_down = self.w_sg = None
+        if limit and not gated:
+            raise ValueError("the clamped unit is a gated one")
+        if groups and (num_experts % groups[0] or not 1 <= groups[1] <= groups[0]):
+            raise ValueError("expert groups: the number of experts must be a multiple of 'count', and 1 <= keep <= count")
+        if groups and groups[1] * (num_experts // groups[0]) < top:
+            raise ValueError("the kept expert groups hold fewer experts than a token chooses")
+        self.rule = dict(renorm=renormalise, scores=scores, groups=tuple(groups) if groups else None, scale=float(scale))
+        self.gated = bool(gated)
+        self.w_router = self.w_gu = self.w_down = self.w_sg = self.w_router_low = None
 
     def children(self) -> List[Part]:
         return [self.shared] if self.shared is not None else []
@@ -50,8 +65,8 @@ class RoutedExperts(FeedForward):
     def param_specs(self) -> List[ParamSpec]:
         specs = [ParamSpec(self.router_name, (self.n_experts, self.hidden), VECTOR)]
         for n in self.expert_names:
-            specs += [ParamSpec(n["gate"], (self.inner, self.hidden), MATRIX),
-                      ParamSpec(n["up"], (self.inner, self.hidden), MATRIX),
+            specs += [ParamSpec(n["gate"], (self.inner, self.hidden), MATRIX)] if self.gated else []
+            specs += [ParamSpec(n["up"], (self.inner, self.hidden), MATRIX),
                       ParamSpec(n["down"], (self.hidden, self.inner), MATRIX)]
         if self.shared is not None and self.shared_gate_name:
             specs.append(ParamSpec(self.shared_gate_name, (1, self.hidden), VECTOR))
@@ -59,22 +74,32 @@ class RoutedExperts(FeedForward):
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.w_router = tensors[self.router_name]
-        # [experts, 2 * inner, hidden]: an expert's gate rows, then its up rows; [experts, hidden, inner]
-        self.w_gu = torch.stack([torch.cat([tensors.pop(n["gate"]), tensors.pop(n["up"])], dim=0)
-                                 for n in self.expert_names]).contiguous()
+        # [experts, 2 * inner, hidden]: an expert's gate rows, then its up rows (up rows alone without a gate);
+        # [experts, hidden, inner]
+        self.w_gu = torch.stack([torch.cat([tensors.pop(n["gate"]), tensors.pop(n["up"])], dim=0) if self.gated
+                                 else tensors.pop(n["up"]) for n in self.expert_names]).contiguous()
+        if self.w_gu.dtype == torch.bfloat16:
+            # bfloat16 factors with float sums give the float router logits exactly: where the stored weights are
+            # bfloat16 numbers, steps of many tokens take their logits from a matrix product
+            self.w_router_low = ops.lossless_bf16(self.w_router)
         self.w_down = torch.stack([tensors.pop(n["down"]) for n in self.expert_names]).contiguous()
         if self.shared is not None and self.shared_gate_name:
             self.w_sg = tensors[self.shared_gate_name].reshape(-1).contiguous()
 
     def forward(self, h: torch.Tensor, ctx: Any) -> Delta:
-        experts, weights, gate = ops.moe_route(h, self.w_router, self.top, ctx.positions, self.w_sg, self.renormalise)
+        if self.w_router_low is not None and self.w_sg is None and h.shape[0] > ROUTE_PRODUCT_MIN_ROWS:
+            z = ops.linear(h, self.w_router_low, out_dtype=torch.float32)
+            experts, weights = ops.moe_choose(z, self.n_experts, self.top, ctx.positions, **self.rule)
+            gate = None
+        else:
+            experts, weights, gate = ops.moe_route(h, self.w_router, self.top, ctx.positions, self.w_sg, **self.rule)
         order = ops.moe_sort(experts, self.n_experts)
         if self.limit is not None:
             # gate | up of every item as the product leaves them, then the clamped unit over the rows
             u = ops.gated_clamped_act(ops.gemm_experts(h, self.w_gu, order, gather=True), None, self.limit, self.alpha,
                                       self.shift)
         else:
-            u = ops.gemm_experts(h, self.w_gu, order, gather=True, gated=True, act=self.activation)
+            u = ops.gemm_experts(h, self.w_gu, order, gather=True, gated=self.gated, act=self.activation)
         y = ops.gemm_experts(u, self.w_down, order, gather=False)
         shared = None
         if self.shared is not None:

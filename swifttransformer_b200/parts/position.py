@@ -70,17 +70,39 @@ class RotaryPairs(PositionEncoding):
     precision and kept as float32; the angle and its sine and cosine are float32 in the kernels.  A mixer that
     prepares its queries and keys in a kernel of its own takes ``inv_freq`` and ``dims`` from here."""
 
-    def __init__(self, dims: int, base: float, **_):
+    neighbours = True
+
+    def __init__(self, dims: int, base: float, scaling: Optional[Dict[str, float]] = None, **_):
+        """``scaling``: None, or {"factor", "original", "fast", "slow"}, the YaRN stretch of the context: with
+        turns(t) = dims * ln(original / (2 pi t)) / (2 ln base), the index at which a pair turns t times within
+        ``original`` positions, pairs before floor(turns(fast)) keep their frequency, those after ceil(turns(slow)) turn
+        ``factor`` times slower, a linear ramp lies between, and sine and cosine are multiplied by
+        0.1 ln(factor) + 1 (``amplitude``)."""
         if dims < 0 or dims % 2:
             raise ValueError(f"rotary dimensions must be even and not negative, got {dims}")
         self.dims, self.base = int(dims), float(base)
+        self.scaling = dict(scaling) if scaling else None
+        self.amplitude = 0.1 * math.log(self.scaling["factor"]) + 1.0 if self.scaling else 1.0
         self._tables: Dict[torch.device, torch.Tensor] = {}
+
+    def frequencies(self) -> List[float]:
+        """One frequency per pair, in double precision."""
+        f = [math.pow(self.base, -2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if not self.scaling:
+            return f
+        s = self.scaling
+        turns = lambda t: self.dims * math.log(s["original"] / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
+        lo, hi = max(math.floor(turns(s["fast"])), 0), min(math.ceil(turns(s["slow"])), self.dims - 1)
+        out = []
+        for i, v in enumerate(f):
+            ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            out.append(v / s["factor"] * ramp + v * (1.0 - ramp))
+        return out
 
     def inv_freq(self, device) -> torch.Tensor:
         device = torch.device(device)
         if device not in self._tables:
-            f = [math.pow(self.base, -2.0 * i / self.dims) for i in range(self.dims // 2)] or [0.0]
-            self._tables[device] = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(device)
+            self._tables[device] = torch.tensor(self.frequencies() or [0.0], dtype=torch.float64).to(torch.float32).to(device)
         return self._tables[device]
 
 
@@ -89,3 +111,5 @@ class RotaryHalves(RotaryPairs):
     """The same rotation with the other pairing: of the first ``dims`` dimensions of a vector, dimension i is paired
     with dimension i + dims/2 (the two halves, not neighbours), i = 0 .. dims/2 - 1, at the angle
     p * base^(-2i/dims).  A mixer that rotates in a kernel of its own takes ``inv_freq`` and ``dims`` from here."""
+
+    neighbours = False
