@@ -13,9 +13,9 @@ single-GPU and exits with 2.
 ``--only decode|prefill`` run one small measurement (for profiling); ``--only mixed`` runs a continuous
 batch of requests of random lengths (prompt portions of 512 tokens beside decoded tokens) through
 ``LLMEngine.generate`` and reports tokens per second, steps and preemptions.  ``--only designs`` measures a
-Fanidra, a Pikadra, a Norelix and a Nafelix model beside an OPT model of equal width, depth and parameter count (prefill, decode,
+Fanidra, a Pikadra, a Norelix, a Nafelix and a Nigilorn model beside an OPT model of equal width, depth and parameter count (prefill, decode,
 and the device time of every operation of one step of each kind; ``--model-name w2048|w4096`` picks one size,
-``--layers`` the depth, ``--designs`` which of the five).
+``--layers`` the depth, ``--designs`` which of the six).
 """
 import argparse
 import json
@@ -113,6 +113,11 @@ def prefill_flops(cfg, n_layers, n):
 # delta rule (the Norelix pair's heads), alternating with gated windowed attention (a window as long as the context);
 # feed-forwards alternate between the dense two-matrix form (inner size one and a half times the gated one's: the
 # same parameter count) and eight clamped experts of half the gated inner size, two per token (the same active count).
+# The Nigilorn model of a size: latent attention with the Pikadra model's sizes (window 512) and a dense gated feed-forward
+# of its size; two layers of selective scan (twice the width in channels, 16 state numbers per channel, a step rank of
+# a sixteenth of the width, four taps) with mixtures of eight two-matrix experts in four groups (three kept), two per
+# token, and a shared expert, each one and a half times as wide as Pikadra's three-matrix ones (the same parameter count);
+# one layer of grouped attention with the Norelix pair's sizes and a window as long as the context.
 DESIGN_SIZES = {
     "w2048": dict(width=2048, opt_heads=32, opt_ffn=8192, heads=16, kv_heads=4, dim=64, vdim=128, ff=5504,
                   rec_heads=16, rec_dim=128, rec_vdim=128, block=512,
@@ -126,14 +131,15 @@ DESIGN_SIZES = {
 
 
 def compare_designs(args, peaks):
-    """Prefill (2048 tokens) and decode (batch 8 behind 512-token prompts) of a Fanidra, a Pikadra, a Norelix, a Nafelix
-    and an OPT model of equal size, random weights, device-timed; and the device time of every operation of one prefill step and one
+    """Prefill (2048 tokens) and decode (batch 8 behind 512-token prompts) of a Fanidra, a Pikadra, a Norelix, a Nafelix, a
+    Nigilorn and an OPT model of equal size, random weights, device-timed; and the device time of every operation of one prefill step and one
     decode step launched kernel by kernel.  One JSON line per (size, design)."""
     import gc
     import numpy as np
     import torch
     from swifttransformer_b200 import ops
-    from swifttransformer_b200.config import FanidraConfig, NafelixConfig, NorelixConfig, OptConfig, PikadraConfig
+    from swifttransformer_b200.config import (FanidraConfig, NafelixConfig, NigilornConfig, NorelixConfig, OptConfig,
+                                              PikadraConfig)
     from swifttransformer_b200.engine.engine import LLMEngine
     from swifttransformer_b200.engine.step import StepEntry
     from swifttransformer_b200.models import random_model
@@ -189,7 +195,21 @@ def compare_designs(args, peaks):
                      for i in range(n_layers)]
         naf = NafelixConfig.from_dict(dict(architecture="Nafelix", vocab=vocab, width=z["width"], streams=4,
                                            norm={"eps": 1e-5}, canon={"taps": 4}, layers=nf_layers))
-        all_designs = {"fanidra": fan, "pikadra": pik, "norelix": nor, "nafelix": naf, "opt": opt}
+        stretch = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+        ng_lat = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": k["ff"]},
+                  "mixer": dict({q: mix[q] for q in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale")}, mask={"size": z["block"]},
+                                rot={"dims": k["rot"], "base": 10000.0, "scaling": stretch})}
+        ng_moe = {"kind": "moe", "expert": {"ff": k["expert_ff"] * 3 // 2}, "shared": {"ff": k["shared_ff"] * 3 // 2},
+                  "router": {"experts": k["experts"], "top": k["top"], "groups": {"count": 4, "keep": 3}, "scale": 2.0}}
+        ng_ssm = {"type": "mamba1", "mlp": ng_moe,
+                  "mixer": dict(inner=2 * z["width"], state=16, dt_rank=z["width"] // 16, conv=4)}
+        ng_att = {"type": "attention", "mlp": ng_moe,
+                  "mixer": dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"], scale=z["dim"] ** -0.5,
+                                mask={"size": 4096}, rot={"dims": z["dim"] // 2, "base": 10000.0, "scaling": stretch})}
+        nig = NigilornConfig.from_dict(dict(architecture="Nigilorn", vocab=vocab, width=z["width"], norm={"eps": 1e-6},
+                                            token_side={"dim": 64}, layers=[(ng_lat, ng_ssm, ng_ssm, ng_att)[i % 4]
+                                                                            for i in range(n_layers)]))
+        all_designs = {"fanidra": fan, "pikadra": pik, "norelix": nor, "nafelix": naf, "nigilorn": nig, "opt": opt}
         return {d: c for d, c in all_designs.items() if not args.designs or d in args.designs.split(",")}
 
     def engine(model, graphs=True):
@@ -292,7 +312,7 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=512)
     ap.add_argument("--layers", type=int, default=0, help="run fewer layers than the model has (0: all)")
     ap.add_argument("--designs", default="", help="with --only designs: which designs to measure, with commas between "
-                    "them (fanidra, pikadra, norelix, nafelix, opt; default: all)")
+                    "them (fanidra, pikadra, norelix, nafelix, nigilorn, opt; default: all)")
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 and prefill measurements")
     ap.add_argument("--no-big", action="store_true", help="skip the OPT-6.7B and OPT-30B points (13 and 60 GB of random weights)")
     ap.add_argument("--launch-floor", action="store_true",

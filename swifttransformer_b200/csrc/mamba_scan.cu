@@ -87,7 +87,7 @@ __device__ __forceinline__ void ms_store_row(float* p, int first, int n, const f
 
 // LOCAL: the scan from a zero state that leaves end state and sum of steps; otherwise the scan that leaves outputs
 template <typename T, int NS, bool LOCAL>
-__global__ void __launch_bounds__(MS_THREADS)
+__global__ void __launch_bounds__(MS_THREADS, NS <= 16 ? 7 : 4)
 mamba_scan_kernel(ScanArgs<T> a) {
     extern __shared__ __align__(16) float ms_smem[];
     const int lpc = a.lpc, nsp = NS * lpc, per_block = MS_THREADS / lpc;

@@ -13,7 +13,7 @@
 //              in `sorted` (item indices), `place[item]` the inverse, and a list of row tiles (expert, first place)
 //              for the grouped products, padded with expert -1.  One block; items of one expert stand in no
 //              particular order, which changes no result: every row of a product is computed on its own.
-// moe_combine: out[t] = sum_k weight[t,k] * y[place[t,k]]  (+ g[t] * shared[t]), in float.
+// moe_combine: out[t] = sum_k weight[t,k] * y[place[t,k]]  (+ g[t] * shared[t], or + shared[t] without gates), in float.
 #include "common.cuh"
 
 #define ROUTE_THREADS 256
@@ -258,7 +258,7 @@ moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ place, const
                 acc = make_float4(fmaf(w, v.x, acc.x), fmaf(w, v.y, acc.y), fmaf(w, v.z, acc.z), fmaf(w, v.w, acc.w));
             }
             if (shared) {
-                const float w = __ldcg(gate + t);
+                const float w = gate ? __ldcg(gate + t) : 1.f;
                 const float4 v = load4_cg(shared + (size_t)t * width + e);
                 acc = make_float4(fmaf(w, v.x, acc.x), fmaf(w, v.y, acc.y), fmaf(w, v.z, acc.z), fmaf(w, v.w, acc.w));
             }
@@ -271,7 +271,7 @@ moe_combine_kernel(const T* __restrict__ y, const int* __restrict__ place, const
             const int p = __ldcg(place + (size_t)t * top + k);
             if (p >= 0) acc = fmaf(__ldcg(weights + (size_t)t * top + k), load1_cg(y + (size_t)p * width + e), acc);
         }
-        if (shared) acc = fmaf(__ldcg(gate + t), load1_cg(shared + (size_t)t * width + e), acc);
+        if (shared) acc = fmaf(gate ? __ldcg(gate + t) : 1.f, load1_cg(shared + (size_t)t * width + e), acc);
         out[(size_t)t * width + e] = from_f32<TO>(acc);
     }
 }

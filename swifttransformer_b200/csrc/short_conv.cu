@@ -22,6 +22,7 @@
 // `conv_state_update`, where one thread per (request, channel) reads all it
 // needs before it writes.
 #include "common.cuh"
+#include <type_traits>
 
 #define CONV_MAX_TAPS 8
 
@@ -129,86 +130,72 @@ conv_state_update_kernel(const TI* __restrict__ in, int ld, float* __restrict__ 
 }
 
 // out[t][c] = act(bias[c] + conv(in)[t][c]);  in: [tokens, ld], its first `channels` columns.  A thread owns V
-// neighbouring channels of TT consecutive tokens of the step and carries the last taps - 1 inputs along in registers:
-// where a request begins (or the thread's first token lies inside one) they are fetched anew, from the step's own rows
-// and, before the step's first token of the request, from its state.  The state is read by several threads and stays
-// as it is (conv_state_update follows), unless `move_state` says that every request brings exactly one token: then the
-// one thread that reads a request's state for a channel also moves it on.
-template <typename T, int V, int TT>
+// neighbouring channels of TT consecutive tokens of the step: its tokens' rows and the K - 1 rows before the first are
+// asked for at once (K: the number of taps, rounded up to 4 or 8; the taps that are not there have weight zero).  Rows
+// from before the step come from the request's state.  Where the thread's tokens belong to several requests it takes
+// them one by one.  The state is read by several threads and stays as it is (conv_state_update follows), unless
+// `move_state` says that every request brings exactly one token: then the one thread that reads a request's state for
+// a channel also moves it on.
+template <typename T, int V, int TT, int K>
 __global__ void __launch_bounds__(128)
 conv_act_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, const float* __restrict__ bias,
                 float* __restrict__ state, T* __restrict__ out, const int* __restrict__ positions,
                 const int* __restrict__ seq_of_token, const int* __restrict__ q_start, const int* __restrict__ slots,
                 int n_tokens, int channels, int taps, int act, int move_state) {
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
-    float wv[V][CONV_MAX_TAPS], bv[V];
+    float wv[V][K], bv[V];
     if (c < channels) {                                 // no kernel writes the filters: fetched before the wait
 #pragma unroll
         for (int v = 0; v < V; ++v) {
             bv[v] = bias ? bias[c + v] : 0.f;
 #pragma unroll
-            for (int j = 0; j < CONV_MAX_TAPS; ++j)     // the newest input's weight stands last, whatever taps is
-                wv[v][j] = j >= CONV_MAX_TAPS - taps ? w[(size_t)(c + v) * taps + j - (CONV_MAX_TAPS - taps)] : 0.f;
+            for (int j = 0; j < K; ++j)                 // the newest input's weight stands last, whatever taps is
+                wv[v][j] = j >= K - taps ? w[(size_t)(c + v) * taps + j - (K - taps)] : 0.f;
         }
     }
     ST_PDL_WAIT();
     ST_PDL_TRIGGER();
     if (c >= channels) return;
-    const int keep = taps - 1;
-    float u[CONV_MAX_TAPS][V];                          // u[CONV_MAX_TAPS - 1 - k]: the input k tokens back
-    int held = -1;                                      // the request whose inputs u holds
-    for (int k = 0; k < TT; ++k) {
-        const int t = blockIdx.x * TT + k;
-        if (t >= n_tokens) return;
-        if (positions[t] < 0) continue;                 // padding token of a fixed-shape step
-        const int b = seq_of_token[t];
+    const int keep = taps - 1, t0 = blockIdx.x * TT;
+    // N tokens from t on, all of request b; u[K - 1 + k]: the input of token t + k
+    auto run = [&](auto n_const, int t, int b) {
+        constexpr int N = decltype(n_const)::value;
+        const int i = t - q_start[b];
         float* st = state + (size_t)slots[b] * keep * channels + c;
-        if (b != held) {
-            held = b;
-            const int i = t - q_start[b];
+        float u[K - 1 + N][V];
 #pragma unroll
-            for (int j = 1; j < CONV_MAX_TAPS; ++j) {
-                float x[V];
+        for (int r = 0; r < K - 1 + N; ++r) {
+            const int back = K - 1 - r;                 // tokens before t (negative: after it)
 #pragma unroll
-                for (int v = 0; v < V; ++v) x[v] = 0.f;
-                if (j <= keep) {
-                    if (j <= i) load_v<V>(in + (size_t)(t - j) * ld + c, x);
-                    else load_v<V>(st + (size_t)(keep + i - j) * channels, x);
-                }
+            for (int v = 0; v < V; ++v) u[r][v] = 0.f;
+            if (back <= i) { if (back <= keep) load_v<V>(in + (size_t)(t - back) * ld + c, u[r]); }
+            else if (back <= keep) load_v<V>(st + (size_t)(keep + i - back) * channels, u[r]);
+        }
 #pragma unroll
-                for (int v = 0; v < V; ++v) u[CONV_MAX_TAPS - 1 - j][v] = x[v];
+        for (int k = 0; k < N; ++k) {
+            float y[V];
+#pragma unroll
+            for (int v = 0; v < V; ++v) {
+                y[v] = bv[v];
+#pragma unroll
+                for (int j = 0; j < K; ++j) y[v] = fmaf(wv[v][j], u[k + j][v], y[v]);
+                y[v] = apply_act(y[v], act);
             }
+            store_v<V>(out + (size_t)(t + k) * channels + c, y);
         }
-        load_v<V>(in + (size_t)t * ld + c, u[CONV_MAX_TAPS - 1]);
-        float y[V];
+        if (N == 1 && move_state) {
 #pragma unroll
-        for (int v = 0; v < V; ++v) {
-            y[v] = bv[v];
-#pragma unroll
-            for (int j = 0; j < CONV_MAX_TAPS; ++j) y[v] = fmaf(wv[v][j], u[j][v], y[v]);
-            y[v] = apply_act(y[v], act);
+            for (int r = 1; r < K; ++r)                 // the oldest kept input stands first
+                if (K - 1 - r < keep) store_v<V>(st + (size_t)(keep - K + r) * channels, u[r]);
         }
-        store_v<V>(out + (size_t)t * channels + c, y);
-        if (move_state) {
-#pragma unroll
-            for (int j = 0; j < CONV_MAX_TAPS - 1; ++j)          // the oldest kept input stands first
-                if (j < keep) {
-                    float x[V];
-#pragma unroll
-                    for (int v = 0; v < V; ++v) {
-                        x[v] = 0.f;
-#pragma unroll
-                        for (int q = 0; q < CONV_MAX_TAPS; ++q)
-                            if (q == CONV_MAX_TAPS - keep + j) x[v] = u[q][v];
-                    }
-                    store_v<V>(st + (size_t)j * channels, x);
-                }
-        }
-#pragma unroll
-        for (int j = 0; j + 1 < CONV_MAX_TAPS; ++j)
-#pragma unroll
-            for (int v = 0; v < V; ++v) u[j][v] = u[j + 1][v];
+    };
+    if (TT > 1 && t0 + TT <= n_tokens && positions[t0] >= 0 && positions[t0 + TT - 1] >= 0 &&
+        seq_of_token[t0] == seq_of_token[t0 + TT - 1]) {
+        run(std::integral_constant<int, TT>{}, t0, seq_of_token[t0]);
+        return;
     }
+    for (int t = t0; t < min(t0 + TT, n_tokens); ++t)
+        if (positions[t] >= 0) run(std::integral_constant<int, 1>{}, t, seq_of_token[t]);      // (else: padding)
 }
 
 ST_EXPORT int st_conv_act(const void* in, int ld, const float* w, const float* bias, float* state, void* out,
@@ -223,7 +210,7 @@ ST_EXPORT int st_conv_act(const void* in, int ld, const float* w, const float* b
     const int tt = n_tokens > 256 ? 8 : 1;              // few tokens: a thread each; many: the inputs are fetched once
     dim3 grid((n_tokens + tt - 1) / tt, (channels + per_block - 1) / per_block);
 #define CA_LAUNCH(T, V, TT)                                                                                              \
-    return st_launch_pdl("conv_act", conv_act_kernel<T, V, TT>, grid, dim3(128), 0, s, (const T*)in, ld, w, bias, state, \
+    return st_launch_pdl("conv_act", taps <= 4 ? conv_act_kernel<T, V, TT, 4> : conv_act_kernel<T, V, TT, 8>, grid, dim3(128), 0, s, (const T*)in, ld, w, bias, state, \
                          (T*)out, positions, seq_of_token, q_start, slots, n_tokens, channels, taps, act, move_state)
 #define CA_PICK(T)                                                                              \
     do {                                                                                        \

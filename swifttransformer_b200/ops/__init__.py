@@ -1210,10 +1210,10 @@ def gemm_experts(a: torch.Tensor, w: torch.Tensor, order: ExpertOrder, gather: b
 
 def moe_combine(y: torch.Tensor, order: ExpertOrder, weights: torch.Tensor, shared: Optional[torch.Tensor] = None,
                 gate: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
-    """out[t] = sum_k weights[t, k] * y[place of (t, k)] (+ gate[t] * shared[t]); sums in float."""
+    """out[t] = sum_k weights[t, k] * y[place of (t, k)] (+ gate[t] * shared[t], ``gate`` None: + shared[t]); sums in float."""
     n, top = weights.shape
     width = y.shape[1]
-    assert y.is_contiguous() and (shared is None or (shared.is_contiguous() and shared.dtype == y.dtype and gate is not None))
+    assert y.is_contiguous() and (shared is None or (shared.is_contiguous() and shared.dtype == y.dtype))
     out = torch.empty((n, width), dtype=out_dtype, device=y.device)
     _check(lib().st_moe_combine(_p(y), _p(order.place), _p(weights), top, _p(shared), _p(gate), n, width, _p(out),
                                 _dt(y), int(out_dtype == torch.float32), _stream()), "moe_combine")

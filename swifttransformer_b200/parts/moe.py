@@ -106,8 +106,6 @@ class RoutedExperts(FeedForward):
             s = self.shared.forward(h, ctx)
             assert s.bias is None and s.parts is None
             shared = s.value
-            if gate is None:
-                gate = torch.ones((h.shape[0],), dtype=torch.float32, device=h.device)
         return Delta(ops.moe_combine(y, order, weights, shared, gate, out_dtype=torch.float32))
 
     def param_bytes(self) -> int:
