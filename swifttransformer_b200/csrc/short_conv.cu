@@ -129,6 +129,32 @@ conv_state_update_kernel(const TI* __restrict__ in, int ld, float* __restrict__ 
     for (int j = 0; j < keep; ++j) st[(size_t)j * channels] = v[j];
 }
 
+// V neighbouring inputs as they stand in memory (asked for early, widened when they are used)
+template <typename T, int V> struct ConvRaw;
+template <> struct ConvRaw<float, 1> {
+    float r;
+    __device__ __forceinline__ void load(const float* p) { r = __ldcg(p); }
+    __device__ __forceinline__ void widen(float* v) const { v[0] = r; }
+};
+template <> struct ConvRaw<bf16, 1> {
+    unsigned short r;
+    __device__ __forceinline__ void load(const bf16* p) { r = __ldcg(reinterpret_cast<const unsigned short*>(p)); }
+    __device__ __forceinline__ void widen(float* v) const { v[0] = __uint_as_float((unsigned)r << 16); }
+};
+template <> struct ConvRaw<float, 4> {
+    float4 r;
+    __device__ __forceinline__ void load(const float* p) { r = __ldcg(reinterpret_cast<const float4*>(p)); }
+    __device__ __forceinline__ void widen(float* v) const { v[0] = r.x; v[1] = r.y; v[2] = r.z; v[3] = r.w; }
+};
+template <> struct ConvRaw<bf16, 4> {
+    uint2 r;
+    __device__ __forceinline__ void load(const bf16* p) { r = __ldcg(reinterpret_cast<const uint2*>(p)); }
+    __device__ __forceinline__ void widen(float* v) const {
+        v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
+        v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
+    }
+};
+
 // out[t][c] = act(bias[c] + conv(in)[t][c]);  in: [tokens, ld], its first `channels` columns.  A thread owns V
 // neighbouring channels of TT consecutive tokens of the step: its tokens' rows and the K - 1 rows before the first are
 // asked for at once (K: the number of taps, rounded up to 4 or 8; the taps that are not there have weight zero).  Rows
@@ -148,6 +174,11 @@ conv_act_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, c
 #pragma unroll
         for (int v = 0; v < V; ++v) {
             bv[v] = bias ? bias[c + v] : 0.f;
+            if (taps == 4 && K == 4) {                  // (a channel's filter is one 16-byte piece)
+                const float4 q = load4(w + (size_t)(c + v) * 4);
+                wv[v][0] = q.x; wv[v][1] = q.y; wv[v][2] = q.z; wv[v][3] = q.w;
+                continue;
+            }
 #pragma unroll
             for (int j = 0; j < K; ++j)                 // the newest input's weight stands last, whatever taps is
                 wv[v][j] = j >= K - taps ? w[(size_t)(c + v) * taps + j - (K - taps)] : 0.f;
@@ -162,10 +193,13 @@ conv_act_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, c
         constexpr int N = decltype(n_const)::value;
         const int i = t - q_start[b];
         float* st = state + (size_t)slots[b] * keep * channels + c;
-        float u[K - 1 + N][V];
+        ConvRaw<T, V> raw[N];
 #pragma unroll
-        for (int r = 0; r < K - 1 + N; ++r) {
-            const int back = K - 1 - r;                 // tokens before t (negative: after it)
+        for (int k = 0; k < N; ++k) raw[k].load(in + (size_t)(t + k) * ld + c);
+        float u[K][V];                                  // the inputs of a token and the K - 1 before it
+#pragma unroll
+        for (int r = 0; r < K - 1; ++r) {
+            const int back = K - 1 - r;                 // tokens before t
 #pragma unroll
             for (int v = 0; v < V; ++v) u[r][v] = 0.f;
             if (back <= i) { if (back <= keep) load_v<V>(in + (size_t)(t - back) * ld + c, u[r]); }
@@ -173,15 +207,21 @@ conv_act_kernel(const T* __restrict__ in, int ld, const float* __restrict__ w, c
         }
 #pragma unroll
         for (int k = 0; k < N; ++k) {
+            raw[k].widen(u[K - 1]);
             float y[V];
 #pragma unroll
             for (int v = 0; v < V; ++v) {
                 y[v] = bv[v];
 #pragma unroll
-                for (int j = 0; j < K; ++j) y[v] = fmaf(wv[v][j], u[k + j][v], y[v]);
+                for (int j = 0; j < K; ++j) y[v] = fmaf(wv[v][j], u[j][v], y[v]);
                 y[v] = apply_act(y[v], act);
             }
             store_v<V>(out + (size_t)(t + k) * channels + c, y);
+            if (N == 1) break;
+#pragma unroll
+            for (int j = 0; j + 1 < K; ++j)
+#pragma unroll
+                for (int v = 0; v < V; ++v) u[j][v] = u[j + 1][v];
         }
         if (N == 1 && move_state) {
 #pragma unroll
