@@ -5,7 +5,7 @@
 //             neighbours, float angle p * freq[i], sincosf); q times the temperature
 //             1 + coef * ln(floor((p + 1) / every) + 1)  (coef == 0: none)
 //   s_j    = scale * q . k_j over the keys the query sees (gqa_attention.cuh: a window of recent keys plus the
-//             first keep_first keys of the request, or all keys up to the query)
+//             first keep_first keys of the request, those of the query's own chunk, or all keys up to the query)
 //   w_j    = exp(s_j) / (sum_i exp(s_i) [+ exp(sink)])
 //   out    = out_scale * (sum_j w_j v_j) [* sigmoid(gate)]
 //
@@ -128,6 +128,140 @@ gqa_prepare_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
             else cache_keys(pool, cache, page, head, pip)[e] = from_f32<T>(x[r] * mult);
         }
     }
+}
+
+// The same with the norm over a whole projection: all query heads' numbers of a token are divided by their common root
+// mean square (eps inside the root) and multiplied by a weight per column, so are all key heads', before the rotation.
+// A block per token: sines and cosines of the token's position once for all heads (shared memory), the two sums of
+// squares in one walk over the row, then queries, keys and values.  VEC: neighbours are paired, and rows, heads and
+// weights allow pieces of four; else one element at a time in either layout.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(GP_THREADS)
+gqa_prepare_whole_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off,
+                              const float* __restrict__ bias, Rotation rot, float temp_coef, int temp_every,
+                              const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                              T* __restrict__ q_out, T* __restrict__ pool, DiffCache cache,
+                              const int* __restrict__ positions, const int* __restrict__ seq_of_token,
+                              const int* __restrict__ slots, const int* __restrict__ block_table, int nh, int write_kv,
+                              int* __restrict__ status) {
+    extern __shared__ float2 turn[];             // [rot.dims / 2] (cosine, sine) times the amplitude
+    __shared__ float scratch[32];
+    ST_PDL_WAIT();
+    ST_PDL_TRIGGER();
+    const int t = blockIdx.x;
+    const int pos = positions[t];
+    if (pos < 0) return;
+    const int dim = cache.kd, vd = cache.vd, nkv = cache.nkv;
+    const int qw = nh * dim, kw = write_kv ? nkv * dim : 0, vw = write_kv ? nkv * vd : 0;
+    int page = -1;
+    if (write_kv) {
+        page = block_table[(size_t)slots[seq_of_token[t]] * cache.max_pages + pos / cache.page_size];
+        if (page < 0 && status && threadIdx.x == 0) *status = 1;
+    }
+    const int pip = pos % cache.page_size;
+    for (int i = threadIdx.x; i < rot.dims / 2; i += GP_THREADS) {
+        float sn, cs;
+        sincosf((float)pos * rot.freq[i], &sn, &cs);
+        turn[i] = make_float2(cs * rot.amp, sn * rot.amp);
+    }
+    const T* row = proj + (size_t)t * ld;
+    auto at = [&](int col) { return load1_cg(row + col) + (bias ? bias[col] : 0.f); };
+    auto at4 = [&](int col) {
+        const float4 v = load4_cg(row + col);
+        return bias ? add4(v, load4(bias + col)) : v;
+    };
+    constexpr int STEP = VEC ? 4 : 1;
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x * STEP; c < qw + kw; c += GP_THREADS * STEP) {
+        const bool is_q = c < qw;
+        const int col = is_q ? q_off + c : k_off + c - qw;
+        float d;
+        if (VEC) {
+            const float4 v = at4(col);
+            d = v.x * v.x + v.y * v.y + (v.z * v.z + v.w * v.w);
+        } else {
+            const float v = at(col);
+            d = v * v;
+        }
+        if (is_q) sq += d; else sk += d;
+    }
+    const float rq = rsqrtf(block_sum(sq, scratch) / (float)qw + eps);       // (its barriers also publish `turn`)
+    const float rk = kw > 0 ? rsqrtf(block_sum(sk, scratch) / (float)kw + eps) : 0.f;
+    const float temp = temp_coef != 0.f ? 1.f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.f) : 1.f;
+    for (int c = threadIdx.x * STEP; c < qw + kw; c += GP_THREADS * STEP) {
+        const bool is_q = c < qw;
+        if (!is_q && page < 0) continue;
+        const int cc = is_q ? c : c - qw, head = cc / dim, e = cc % dim;
+        const int col = (is_q ? q_off : k_off) + cc;
+        const float* w = is_q ? q_w : k_w;
+        const float r = is_q ? rq : rk;
+        T* dst = is_q ? q_out + (size_t)t * qw + cc : cache_keys(pool, cache, page, head, pip) + e;
+        if (VEC) {
+            const float4 v = at4(col), g = load4(w + cc);
+            float4 y = make_float4(v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w);
+            if (e < rot.dims) {
+                const float2 a = turn[e >> 1];
+                y = make_float4(y.x * a.x - y.y * a.y, y.y * a.x + y.x * a.y, y.z, y.w);
+            }
+            if (e + 2 < rot.dims) {
+                const float2 a = turn[(e >> 1) + 1];
+                y = make_float4(y.x, y.y, y.z * a.x - y.w * a.y, y.w * a.x + y.z * a.y);
+            }
+            if (is_q) y = make_float4(y.x * temp, y.y * temp, y.z * temp, y.w * temp);
+            store4(dst, y);
+        } else {
+            float y = at(col) * r * w[cc];
+            if (e < rot.dims) {
+                const int partner = rot_partner(rot, e);
+                const int half = rot.dims >> 1;
+                const bool low = rot.neighbours ? !(e & 1) : e < half;
+                const float2 a = turn[rot.neighbours ? (e >> 1) : (low ? e : e - half)];
+                const float z = at(col - e + partner) * r * w[cc - e + partner];
+                y = low ? y * a.x - z * a.y : y * a.x + z * a.y;
+            }
+            *dst = from_f32<T>(is_q ? y * temp : y);
+        }
+    }
+    if (page < 0) return;
+    for (int c = threadIdx.x * STEP; c < vw; c += GP_THREADS * STEP) {
+        T* dst = cache_values(pool, cache, page, c / vd, pip) + c % vd;
+        if (VEC) store4(dst, at4(v_off + c));
+        else *dst = from_f32<T>(at(v_off + c));
+    }
+}
+
+// q_w [nh * dim], k_w [nkv * dim] float: the norms' weights; v_off may be k_off (values that are the keys as projected)
+ST_EXPORT int st_gqa_prepare_whole_norm(const void* proj, int ld, int q_off, int k_off, int v_off, const float* bias,
+                                        const float* inv_freq, int rot_dims, int neighbours, float rot_amp,
+                                        float temp_coef, int temp_every, const float* q_w, const float* k_w, float eps,
+                                        void* q_out, void* pool, long long page_stride, long long entry_offset,
+                                        const int* positions, const int* seq_of_token, const int* slots,
+                                        const int* block_table, int max_pages, int n_tokens, int nh, int nkv, int dim,
+                                        int vd, int page_size, int write_kv, int* status, int dtype, void* stream) {
+    if (n_tokens <= 0) return 0;
+    if (nh <= 0 || nkv <= 0 || nh % nkv || dim <= 0 || vd <= 0 || page_size <= 0 || !q_w || !k_w) return ST_ERR_BAD_ARG;
+    if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims > 0 && !inv_freq)) return ST_ERR_BAD_ARG;
+    if (temp_coef != 0.f && temp_every <= 0) return ST_ERR_BAD_ARG;
+    if (rot_dims > 8192) return ST_ERR_TOO_LARGE;
+    const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
+    const Rotation rot = {inv_freq, rot_dims, neighbours, rot_amp};
+    const size_t smem = (size_t)(rot_dims / 2) * sizeof(float2);
+    const bool vec = (neighbours || rot_dims == 0) && dim % 4 == 0 && vd % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 &&
+                     k_off % 4 == 0 && v_off % 4 == 0 && page_stride % 4 == 0 && entry_offset % 4 == 0 && aligned16(proj) &&
+                     aligned16(bias) && aligned16(q_w) && aligned16(k_w) && aligned16(q_out) && aligned16(pool);
+    cudaStream_t s = (cudaStream_t)stream;
+#define GW_LAUNCH(T, VEC)                                                                                                 \
+    return st_launch_pdl("gqa_prepare", gqa_prepare_whole_norm_kernel<T, VEC>, dim3(n_tokens), dim3(GP_THREADS), smem, s, \
+                         (const T*)proj, ld, q_off, k_off, v_off, bias, rot, temp_coef, temp_every, q_w, k_w, eps,        \
+                         (T*)q_out, (T*)pool, c, positions, seq_of_token, slots, block_table, nh, write_kv, status)
+    if (dtype == 0) {
+        if (vec) GW_LAUNCH(float, true);
+        GW_LAUNCH(float, false);
+    }
+    if (dtype != 1) return ST_ERR_BAD_DTYPE;
+    if (vec) GW_LAUNCH(bf16, true);
+    GW_LAUNCH(bf16, false);
+#undef GW_LAUNCH
 }
 
 ST_EXPORT int st_gqa_prepare(const void* proj, int ld, int q_off, int k_off, int v_off, const float* bias,
@@ -275,12 +409,12 @@ ST_EXPORT int st_gqa_attention_plain(const void* q, const void* pool, long long 
                                      const int* slots, const int* block_table, int max_pages, int n_tokens, int nh,
                                      int nkv, int dim, int vd, int page_size, float scale, int window, int keep_first,
                                      int has_sink, float sink, const void* gate, long long gate_ld, float out_scale,
-                                     int* status, int dtype, void* stream, const float* sinks, int gate_heads) {
+                                     int* status, int dtype, void* stream, const float* sinks, int gate_heads, int chunk) {
     if (n_tokens <= 0) return 0;
-    if (nh <= 0 || nkv <= 0 || nh % nkv || dim <= 0 || vd <= 0 || page_size <= 0 || keep_first < 0) return ST_ERR_BAD_ARG;
+    if (nh <= 0 || nkv <= 0 || nh % nkv || dim <= 0 || vd <= 0 || page_size <= 0 || keep_first < 0 || chunk < 0) return ST_ERR_BAD_ARG;
     if (vd > G_VPASS * GK || dim > 4096) return ST_ERR_TOO_LARGE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
-    const GqaMask mask = {window, keep_first};
+    const GqaMask mask = {window, keep_first, chunk};
     const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr, gate_heads};
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(n_tokens, nh);
@@ -561,12 +695,12 @@ ST_EXPORT int st_gqa_attention_single(const void* q, const void* pool, long long
                                       const int* slots, const int* block_table, int max_pages, int n_tokens, int nh,
                                       int nkv, int dim, int vd, int page_size, float scale, int window, int keep_first,
                                       int has_sink, float sink, const void* gate, long long gate_ld, float out_scale,
-                                      int* status, void* stream, const float* sinks, int gate_heads) {
+                                      int* status, void* stream, const float* sinks, int gate_heads, int chunk) {
     if (n_tokens <= 0) return 0;
-    if (page_size <= 0 || keep_first < 0) return ST_ERR_BAD_ARG;
+    if (page_size <= 0 || keep_first < 0 || chunk < 0) return ST_ERR_BAD_ARG;
     if (!st_gqa_attention_single_applies(nh, nkv, dim, vd)) return ST_ERR_BAD_SIZE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
-    const GqaMask mask = {window, keep_first};
+    const GqaMask mask = {window, keep_first, chunk};
     const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr, gate_heads};
     cudaStream_t s = (cudaStream_t)stream;
     // Query heads per block: the whole group when that gives blocks for three quarters of the device (a key or value

@@ -5,8 +5,8 @@
 // memory, filled by 16-byte asynchronous copies from the pages (two stages: the next tile lands while this one
 // is multiplied).  Each warp keeps S = Q K^T, the running maximum and sum and O = P V (16 x vd) in registers.
 //
-// Mask (gqa_attention.cuh): with a window the keys a block reads are two runs of tiles, those that hold the kept
-// first keys of the request and those from the window of the block's first row up to its last row; the tiles
+// Mask (gqa_attention.cuh): with a window or chunks the keys a block reads are two runs of tiles, those that hold the kept
+// first keys of the request and those from the first key of the block's first row up to its last row; the tiles
 // between them are never touched (their pages may be gone).  A tile wholly inside the range of every row of a
 // warp takes no mask.  The softmax's extra term joins the sum once, after the last tile.  The head's result is
 // multiplied by out_scale and, with a gate, by sigmoid(gate logit) when it is stored.
@@ -89,21 +89,23 @@ gqa_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__ 
     const int rows_here = min(GT_ROWS, n_new - off);
     const int p_first = start + off, hi = p_first + rows_here - 1;
     const int lo = gqa_lo(p_first, mask);
-    const int keep = mask.window > 0 ? mask.keep_first : 0;
+    const bool limited = gqa_limited(mask);
+    const int keep = mask.keep_first;
 
     // this thread's two query rows (g and g + 8 of the warp's sixteen)
-    int pos[2];
+    int pos[2], row_lo[2];
     bool live[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         const int row = row0 + g + 8 * r;
         live[r] = row < rows_here;
         pos[r] = p_first + row;
+        row_lo[r] = gqa_lo(pos[r], mask);
     }
     // what decides whether a key tile needs a mask for this warp's sixteen rows
     const bool w_all_live = row0 + 15 < rows_here;
     const bool w_any_live = row0 < rows_here;
-    const int w_pos_min = p_first + row0, w_lo_max = gqa_lo(p_first + row0 + 15, mask);
+    const int w_pos_min = p_first + row0, w_lo_min = gqa_lo(w_pos_min, mask), w_lo_max = gqa_lo(w_pos_min + 15, mask);
     // Q fragments, from global memory (once)
     uint32_t qa[DIMT / 16][4];
 #pragma unroll
@@ -150,7 +152,7 @@ gqa_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__ 
         // a warp that has no rows, whose rows all lie before the tile's first key, or whose rows' windows all start
         // behind the tile's last key (and the tile holds no kept key) has nothing to do with it
         if (w_any_live && key0 <= min(p_first + row0 + 15, hi) &&
-            !(mask.window > 0 && key0 >= keep && key0 + GT_KEYS - 1 < gqa_lo(w_pos_min, mask))) {
+            !(limited && key0 >= keep && key0 + GT_KEYS - 1 < w_lo_min)) {
             // S = Q K^T for the tile's 64 keys
             float s[GT_KEYS / 8][4];
 #pragma unroll
@@ -167,7 +169,7 @@ gqa_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__ 
             }
             float tmax[2] = {-INFINITY, -INFINITY};
             const bool inside = w_all_live && key0 + GT_KEYS - 1 <= w_pos_min &&
-                                (mask.window <= 0 || key0 >= w_lo_max || key0 + GT_KEYS <= keep);
+                                (key0 >= w_lo_max || key0 + GT_KEYS <= keep);
             if (inside) {
 #pragma unroll
                 for (int nt = 0; nt < GT_KEYS / 8; ++nt)
@@ -183,7 +185,7 @@ gqa_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__ 
 #pragma unroll
                     for (int x = 0; x < 4; ++x) {
                         const int r = x >> 1, key = key0 + nt * 8 + 2 * tq + (x & 1);
-                        const float v = (live[r] && gqa_seen(key, pos[r], mask)) ? s[nt][x] * scale_l2 : -INFINITY;
+                        const float v = (live[r] && gqa_seen(key, pos[r], row_lo[r], mask)) ? s[nt][x] * scale_l2 : -INFINITY;
                         s[nt][x] = v;
                         tmax[r] = fmaxf(tmax[r], v);
                     }
@@ -308,13 +310,13 @@ ST_EXPORT int st_gqa_attention_tiles(const void* q, const void* pool, long long 
                                      const int* start_pos, const int* slots, const int* block_table, int max_pages,
                                      int nh, int nkv, int dim, int vd, int page_size, float scale, int window,
                                      int keep_first, int has_sink, float sink, const void* gate, long long gate_ld,
-                                     float out_scale, int* status, void* stream, const float* sinks, int gate_heads) {
+                                     float out_scale, int* status, void* stream, const float* sinks, int gate_heads, int chunk) {
     if (n_tiles <= 0) return 0;
-    if (nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || tile_rows <= 0 || keep_first < 0) return ST_ERR_BAD_ARG;
+    if (nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || tile_rows <= 0 || keep_first < 0 || chunk < 0) return ST_ERR_BAD_ARG;
     if (!st_gqa_attention_tiles_applies(dim, vd)) return ST_ERR_BAD_SIZE;
     if (gate && !gate_heads && ((gate_ld & 1) || ((uintptr_t)gate & 3))) return ST_ERR_BAD_ARG;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
-    const GqaMask mask = {window, keep_first};
+    const GqaMask mask = {window, keep_first, chunk};
     const GqaEpilogue epi = {gate, gate_ld, out_scale, has_sink ? sinks : nullptr, gate_heads};
     cudaStream_t s = (cudaStream_t)stream;
 #define GT_ARGS q, pool, c, out, tiles, n_tiles, tile_rows, q_start, start_pos, slots, block_table, nh, scale, mask, has_sink, \

@@ -168,7 +168,7 @@ ST_EXPORT int st_talk_attention_plain(const void* q, const void* pool, long long
     const size_t smem = ((size_t)nh * dim + 2 * (size_t)nh * TK + (size_t)nh * nh + 2 * (size_t)nh) * sizeof(float);
     if (smem > 200 * 1024) return ST_ERR_TOO_LARGE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
-    const GqaMask mask = {window, keep_first};
+    const GqaMask mask = {window, keep_first, 0};
     const GqaEpilogue epi = {gate, gate_ld, out_scale, sinks};
     cudaStream_t s = (cudaStream_t)stream;
 #define TALK_PLAIN(T)                                                                                                 \

@@ -259,7 +259,7 @@ ST_EXPORT int st_talk_attention_single(const void* q, const void* pool, long lon
     if (page_size <= 0 || keep_first < 0 || !scratch) return ST_ERR_BAD_ARG;
     if (!st_talk_attention_single_applies(nh, nkv, dim, vd, n_cap)) return ST_ERR_BAD_SIZE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
-    const GqaMask mask = {window, keep_first};
+    const GqaMask mask = {window, keep_first, 0};
     const GqaEpilogue epi = {gate, gate_ld, out_scale, sinks};
     cudaStream_t s = (cudaStream_t)stream;
     const int rep = nh / nkv;

@@ -103,12 +103,13 @@ talk_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__
     const int p_first = start + off, hi = p_first + rows_here - 1;
     const int lo = gqa_lo(p_first, mask);
     const int keep = mask.window > 0 ? mask.keep_first : 0;
-    int pos[2];
+    int pos[2], row_lo[2];
     bool live[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         live[r] = g + 8 * r < rows_here;
         pos[r] = p_first + g + 8 * r;
+        row_lo[r] = gqa_lo(pos[r], mask);
     }
     // the queries of this warp's heads (head warp + 8 i), as row operands
     uint32_t qa[HPW][DIMT / 16][4];
@@ -161,7 +162,7 @@ talk_attention_tiles_kernel(const bf16* __restrict__ q, const bf16* __restrict__
 #pragma unroll
                 for (int x = 0; x < 4; ++x) {
                     const int r = x >> 1, key = key0 + nt * 8 + 2 * tq + (x & 1);
-                    s[nt][x] = (live[r] && gqa_seen(key, pos[r], mask)) ? s[nt][x] * scale_l2 : -INFINITY;
+                    s[nt][x] = (live[r] && gqa_seen(key, pos[r], row_lo[r], mask)) ? s[nt][x] * scale_l2 : -INFINITY;
                 }
             }
         }
@@ -406,7 +407,7 @@ ST_EXPORT int st_talk_attention_tiles(const void* q, const void* pool, long long
     if (page_size <= 0 || keep_first < 0 || tile_rows <= 0 || tile_rows % TT_ROWS) return ST_ERR_BAD_ARG;
     if (!st_talk_attention_tiles_applies(nh, nkv, dim, vd)) return ST_ERR_BAD_SIZE;
     const DiffCache c = {max_pages, page_size, nkv, dim, vd, page_stride, entry_offset};
-    const GqaMask mask = {window, keep_first};
+    const GqaMask mask = {window, keep_first, 0};
     const GqaEpilogue epi = {gate, gate_ld, out_scale, sinks};
     cudaStream_t s = (cudaStream_t)stream;
     int v_parts, warps, hpw;

@@ -132,7 +132,8 @@ class CausalLM:
         self.embedding, self.position = model_def.embedding, model_def.position
         self.blocks, self.layer_order = model_def.blocks, model_def.layer_order
         self.final_norm, self.head = model_def.final_norm, model_def.head
-        self._keeps_embedding = any(getattr(b, "wants_embedding", False) for b in self.blocks)
+        wanted = {getattr(b, "wants_embedding", False) for b in self.blocks}
+        self._keeps_embedding, self._keeps_embedded = True in wanted, "float" in wanted
         # a hook for tools that look at the residual stream: called with (layer step index, stream) after every step
         self.after_layer: Optional[Callable[[int, Any], None]] = None
 
@@ -168,6 +169,8 @@ class CausalLM:
             # a copy in the activation type: the layers change x in place
             stream.x0 = stream.materialise()
             stream.act = None
+        if self._keeps_embedded:
+            stream.embedded = x.clone()
         nvtx = getattr(ctx, "nvtx", False)
         for i, st in enumerate(self.layer_order):
             if nvtx:
@@ -181,6 +184,11 @@ class CausalLM:
                 torch.cuda.nvtx.range_pop()
         if ctx.n_want == 0:
             return None
+        if stream.scaled_pending is not None and self.final_norm is not None and self.final_norm.kind == "rmsnorm":
+            # the last block's sum and the final norm of the wanted rows alone, in one kernel
+            h = torch.empty((ctx.want_rows.numel(), x.shape[1]), dtype=self.dtype, device=x.device)
+            stream.settle_scaled(None, self.final_norm, h, rows=ctx.want_rows)
+            return self.head.forward(h)
         stream.fold()
         if self.final_norm is not None:
             h = self.final_norm.apply(stream.x, stream.pending, act_dtype=self.dtype, rows=ctx.want_rows)

@@ -1123,34 +1123,43 @@ def _grouped_mma(a: torch.Tensor, k_dim: int, lda: int, a_goff: int, w_gstride: 
                                                        ctypes.c_longlong(w_gstride))))
 
 
-def _route_rule(scores: str, groups, renorm: bool, scale: float):
+def _route_rule(scores: str, groups, renorm: bool, scale: float, correction: Optional[torch.Tensor], group_score: str,
+                n_experts: int):
+    if group_score not in ("top2", "max"):
+        raise KernelError(f"a group's score is 'top2' or 'max', not {group_score!r}")
+    if correction is not None:
+        assert correction.dtype == torch.float32 and correction.numel() == n_experts and correction.is_contiguous()
     if scores not in ("softmax", "sigmoid"):
         raise KernelError(f"router scores are 'softmax' or 'sigmoid', not {scores!r}")
     count, keep = groups if groups else (0, 0)
-    return int(scores == "sigmoid"), int(count), int(keep), int(renorm), _f(scale)
+    return int(scores == "sigmoid"), int(count), int(keep), int(renorm), _f(scale), _p(correction), int(group_score == "max")
 
 
 def moe_choose(logits: torch.Tensor, n_experts: int, top: int, positions: Optional[torch.Tensor] = None,
-               renorm: bool = False, scores: str = "softmax", groups: Optional[Sequence[int]] = None, scale: float = 1.0):
+               renorm: bool = False, scores: str = "softmax", groups: Optional[Sequence[int]] = None, scale: float = 1.0,
+               correction: Optional[torch.Tensor] = None, group_score: str = "top2"):
     """The choice of ``moe_route`` alone, from float32 router logits [tokens, >= n_experts] that a product left."""
     n = logits.shape[0]
     assert logits.dtype == torch.float32 and logits.is_contiguous() and logits.shape[1] >= n_experts
     experts = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
-    _check(lib().st_moe_choose(_p(logits), logits.shape[1], n, n_experts, top, *_route_rule(scores, groups, renorm, scale),
-                               _p(positions), _p(experts), _p(weights), _stream()), "moe_choose")
+    _check(lib().st_moe_choose(_p(logits), logits.shape[1], n, n_experts, top,
+                               *_route_rule(scores, groups, renorm, scale, correction, group_score, n_experts), _p(positions), _p(experts), _p(weights), _stream()), "moe_choose")
     return experts, weights
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, positions: Optional[torch.Tensor] = None,
               w_gate: Optional[torch.Tensor] = None, renorm: bool = False, scores: str = "softmax",
-              groups: Optional[Sequence[int]] = None, scale: float = 1.0):
+              groups: Optional[Sequence[int]] = None, scale: float = 1.0, correction: Optional[torch.Tensor] = None,
+              group_score: str = "top2"):
     """-> (experts int32 [tokens, top], weights float [tokens, top], gate float [tokens] or None).  Router logits,
     softmax over all experts and the choice in float; ``w_router`` float [experts, width]; ``w_gate`` float [width]:
     also sigmoid(w_gate . h) per token.  Tokens at a negative position get expert -1.  ``scores`` "sigmoid": the scores
     are sigmoids of the logits.  ``groups`` (count, keep): the experts form ``count`` equal groups of neighbours, only the
     ``keep`` with the largest sums of their two largest scores can be chosen from.  The weights (divided by their sum
-    with ``renorm``) are multiplied by ``scale``."""
+    with ``renorm``) are multiplied by ``scale``.  ``correction`` float [experts]: experts (and groups) are chosen by
+    score + correction, the weights stay the bare scores.  ``group_score`` "max": a group counts by its largest choice
+    score alone."""
     n, width = h.shape
     assert h.is_contiguous() and w_router.dtype == torch.float32 and w_router.is_contiguous() and w_router.shape[1] == width
     experts = torch.empty((n, top), dtype=torch.int32, device=h.device)
@@ -1159,7 +1168,7 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, top: int, positions: Opti
     if w_gate is not None:
         assert w_gate.dtype == torch.float32 and w_gate.numel() == width and w_gate.is_contiguous()
     _check(lib().st_moe_route(_p(h), n, width, _p(w_router), w_router.shape[0], top,
-                              *_route_rule(scores, groups, renorm, scale), _p(w_gate),
+                              *_route_rule(scores, groups, renorm, scale, correction, group_score, w_router.shape[0]), _p(w_gate),
                               _p(positions), _p(experts), _p(weights), _p(gate), _dt(h), _stream()), "moe_route")
     return experts, weights, gate
 
@@ -1209,15 +1218,75 @@ def gemm_experts(a: torch.Tensor, w: torch.Tensor, order: ExpertOrder, gather: b
 
 
 def moe_combine(y: torch.Tensor, order: ExpertOrder, weights: torch.Tensor, shared: Optional[torch.Tensor] = None,
-                gate: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
-    """out[t] = sum_k weights[t, k] * y[place of (t, k)] (+ gate[t] * shared[t], ``gate`` None: + shared[t]); sums in float."""
+                gate: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.float32,
+                identity: Optional[torch.Tensor] = None, experts: Optional[torch.Tensor] = None,
+                n_real: int = 0) -> torch.Tensor:
+    """out[t] = sum_k weights[t, k] * y[place of (t, k)] (+ gate[t] * shared[t], ``gate`` None: + shared[t]); sums in float.
+    ``identity`` [tokens, width]: choices of ``experts`` (int32 [tokens, top]) at or above ``n_real`` give their weight
+    times the token's row of it."""
     n, top = weights.shape
     width = y.shape[1]
     assert y.is_contiguous() and (shared is None or (shared.is_contiguous() and shared.dtype == y.dtype))
     out = torch.empty((n, width), dtype=out_dtype, device=y.device)
-    _check(lib().st_moe_combine(_p(y), _p(order.place), _p(weights), top, _p(shared), _p(gate), n, width, _p(out),
+    if identity is not None:
+        assert identity.is_contiguous() and identity.dtype == y.dtype and identity.shape == (n, width)
+        assert experts.dtype == torch.int32 and experts.is_contiguous() and experts.shape == (n, top)
+    _check(lib().st_moe_combine(_p(y), _p(order.place), _p(weights), top, _p(shared), _p(gate), _p(experts), n_real,
+                                _p(identity), n, width, _p(out),
                                 _dt(y), int(out_dtype == torch.float32), _stream()), "moe_combine")
     return out
+
+
+class ExpertSum:
+    """A mixture's result before it is summed: the experts' rows in sorted order with what the sum needs, for kernels
+    that form it where they read it (``scaled_sum_norms``); ``total`` forms it (float32)."""
+
+    def __init__(self, y: torch.Tensor, order: ExpertOrder, weights: torch.Tensor, experts: Optional[torch.Tensor] = None,
+                 n_real: int = 0, identity: Optional[torch.Tensor] = None):
+        self.y, self.order, self.weights, self.experts, self.n_real, self.identity = y, order, weights, experts, n_real, identity
+
+    def total(self) -> torch.Tensor:
+        return moe_combine(self.y, self.order, self.weights, identity=self.identity, experts=self.experts, n_real=self.n_real)
+
+
+def scaled_sum_norms(x: torch.Tensor, eps: float, a: Optional[torch.Tensor] = None, a_scale: Optional[torch.Tensor] = None,
+                     f: Optional[torch.Tensor] = None, f_scale: Optional[torch.Tensor] = None,
+                     e: Optional[torch.Tensor] = None, items: Optional[ExpertSum] = None,
+                     gain1: Optional[torch.Tensor] = None, out1: Optional[torch.Tensor] = None,
+                     gain2: Optional[torch.Tensor] = None, out2: Optional[torch.Tensor] = None,
+                     positions: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> None:
+    """x <- v = x + e + (a_scale * a + f_scale * f) in place on the float32 residual rows, and out1 / out2 = v / sqrt(mean(v^2)
+    + eps) * gain1 / gain2 in their type, in one pass; each of e, a, f (float32 [rows, width]; the scales float32 [width])
+    may be absent.  ``items``: f is the sum of a mixture's experts, formed here.  ``rows`` (int32): only these rows are
+    read, x stays as it is, and the outputs stand in their order.  Rows at a negative position are left alone."""
+    width = x.shape[1]
+    n = rows.numel() if rows is not None else x.shape[0]
+    assert x.dtype == torch.float32 and x.is_contiguous() and not (items is not None and f is not None)
+    for t in (e, a, f):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == x.shape)
+    for g in (a_scale, f_scale, gain1, gain2):
+        assert g is None or (g.dtype == torch.float32 and g.is_contiguous() and g.numel() == width)
+    code = None
+    for o in (out1, out2):
+        assert o is None or (o.is_contiguous() and o.shape == (n, width))
+        code = _dt(o) if o is not None else code
+    y = place = weights = experts = identity = None
+    top = n_real = 0
+    if items is not None:
+        y, place, weights, top = items.y, items.order.place, items.weights, items.weights.shape[1]
+        experts, identity, n_real = items.experts, items.identity, items.n_real
+        assert y.is_contiguous() and y.shape[1] == width and weights.shape[0] == x.shape[0] and (code is None or _dt(y) == code)
+        assert identity is None or (identity.is_contiguous() and identity.dtype == y.dtype and identity.shape == x.shape)
+        code = _dt(y)
+    _check(lib().st_scaled_sum_norms(_p(x), _p(a), _p(a_scale), _p(f), _p(f_scale), _p(e), _p(y), _p(place), _p(weights),
+                                     _p(experts), top, n_real, _p(identity), _p(gain1), _p(gain2), _f(eps), _p(rows), n, width,
+                                     _p(positions), _p(out1), _p(out2), code if code is not None else 0, _stream()),
+           "scaled_sum_norms")
+
+
+def scaled_sum_norms_max_top() -> int:
+    """The most choices per token whose experts ``scaled_sum_norms`` sums itself."""
+    return int(lib().st_scaled_sum_norms_max_top())
 
 
 def concat_rows(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
@@ -1300,6 +1369,31 @@ def gqa_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias: Op
                                 _f(norm_eps), int(neighbours), _f(rot_amp)), "gqa_prepare")
 
 
+def gqa_prepare_whole_norm(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias: Optional[torch.Tensor],
+                           inv_freq: Optional[torch.Tensor], rot_dims: int, temp_coef: float, temp_every: int,
+                           q_out: torch.Tensor, pool: torch.Tensor, layer: int, positions: torch.Tensor,
+                           seq_of_token: torch.Tensor, slots: torch.Tensor, block_table: torch.Tensor, nh: int, nkv: int,
+                           dim: int, vd: int, page_size: int, status: Optional[torch.Tensor], q_norm: torch.Tensor,
+                           k_norm: torch.Tensor, eps: float, write_kv: bool = True, neighbours: bool = False,
+                           rot_amp: float = 1.0) -> None:
+    """``gqa_prepare`` with the norm over whole projections: before the rotation all the query heads' numbers of a token
+    are divided by their common root mean square (``eps`` inside the root) and multiplied by ``q_norm`` [nh * dim]
+    (float32), all the key heads' likewise with ``k_norm`` [nkv * dim]; biases come first.  The values are the columns
+    from v_off on plus their bias; v_off = k_off: the values are the keys as projected."""
+    assert proj.is_contiguous() and q_out.is_contiguous() and q_out.shape == (proj.shape[0], nh * dim)
+    assert proj.dtype == q_out.dtype == pool.dtype
+    assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.numel() == nh * dim and k_norm.numel() == nkv * dim
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.numel() == proj.shape[1]
+    stride, off = _gqa_pool(pool, layer, nkv, dim, vd, page_size)
+    _check(lib().st_gqa_prepare_whole_norm(_p(proj), proj.shape[1], q_off, k_off, v_off, _p(bias), _p(inv_freq), rot_dims,
+                                           int(neighbours), _f(rot_amp), _f(temp_coef), temp_every, _p(q_norm), _p(k_norm),
+                                           _f(eps), _p(q_out), _p(pool), stride, off, _p(positions), _p(seq_of_token),
+                                           _p(slots), _p(block_table), block_table.shape[1], proj.shape[0], nh, nkv, dim,
+                                           vd, page_size, int(write_kv), _p(status), _dt(proj), _stream()),
+           "gqa_prepare_whole_norm")
+
+
 def _sink_args(sink, nh: int):
     """(has_sink, the one logit, the logits per head): ``sink`` is None, a number, or a float32 tensor [heads]."""
     if sink is None:
@@ -1324,12 +1418,14 @@ def gqa_attention_plain(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                         dim: int, vd: int, page_size: int, scale: float, window: int, keep_first: int,
                         sink: Optional[float], gate: Optional[torch.Tensor], gate_off: int, out_scale: float,
                         status: Optional[torch.Tensor] = None, items: Optional[torch.Tensor] = None,
-                        n_items: Optional[int] = None, gate_heads: bool = False) -> torch.Tensor:
+                        n_items: Optional[int] = None, gate_heads: bool = False, chunk: int = 0) -> torch.Tensor:
     """Grouped attention of every token of the step (or of those ``items`` lists) over the paged cache, in float
     arithmetic for either storage type.  ``window`` 0: all keys up to the query; else the last ``window`` keys and
     the request's first ``keep_first``.  ``sink``: a logit that joins the softmax's denominator (None: none).
     ``gate`` [tokens, columns]: the head's result is multiplied by sigmoid of its columns from ``gate_off`` on.
-    ``sink`` may also be a float32 tensor [heads]: a logit per head.  ``gate_heads``: one gate column per head."""
+    ``sink`` may also be a float32 tensor [heads]: a logit per head.  ``gate_heads``: one gate column per head.
+    ``chunk`` > 0: of the keys a query would see otherwise, only those of its own run of ``chunk`` positions, counted
+    from position 0 (and the kept first ones)."""
     assert q.is_contiguous() and out.is_contiguous() and out.shape == (q.shape[0], nh * vd)
     stride, off, gate_ptr, gate_ld = _gqa_tail(pool, layer, nkv, dim, vd, page_size, scale, window, keep_first, sink,
                                                gate, gate_off, out_scale)
@@ -1339,7 +1435,7 @@ def gqa_attention_plain(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                                         _p(seq_of_token), _p(slots), _p(block_table), block_table.shape[1], n, nh, nkv,
                                         dim, vd, page_size, _f(scale), window, keep_first, has_sink,
                                         sink_one, gate_ptr, gate_ld, _f(out_scale), _p(status), _dt(q),
-                                        _stream(), sinks, int(gate_heads)), "gqa_attention_plain")
+                                        _stream(), sinks, int(gate_heads), chunk), "gqa_attention_plain")
     return out
 
 
@@ -1414,7 +1510,7 @@ def gqa_attention_tiles(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                         slots: torch.Tensor, block_table: torch.Tensor, nh: int, nkv: int, dim: int, vd: int,
                         page_size: int, scale: float, window: int, keep_first: int, sink: Optional[float],
                         gate: Optional[torch.Tensor], gate_off: int, out_scale: float,
-                        status: Optional[torch.Tensor] = None, gate_heads: bool = False) -> torch.Tensor:
+                        status: Optional[torch.Tensor] = None, gate_heads: bool = False, chunk: int = 0) -> torch.Tensor:
     """The same attention for tiles of ``tile_rows`` query rows (tiles: int32 [n_tiles, 2] = request of the step,
     offset of the tile among its new tokens) on the warp-level tensor cores, bfloat16 only."""
     if not (q.dtype == torch.bfloat16 and bool(lib().st_gqa_attention_tiles_applies(dim, vd))):
@@ -1427,7 +1523,7 @@ def gqa_attention_tiles(q: torch.Tensor, pool: torch.Tensor, layer: int, out: to
                                         _p(q_start), _p(start_pos), _p(slots), _p(block_table), block_table.shape[1],
                                         nh, nkv, dim, vd, page_size, _f(scale), window, keep_first,
                                         has_sink, sink_one, gate_ptr, gate_ld, _f(out_scale),
-                                        _p(status), _stream(), sinks, int(gate_heads)), "gqa_attention_tiles")
+                                        _p(status), _stream(), sinks, int(gate_heads), chunk), "gqa_attention_tiles")
     return out
 
 
@@ -1436,7 +1532,7 @@ def gqa_attention_single(q: torch.Tensor, pool: torch.Tensor, layer: int, out: t
                          dim: int, vd: int, page_size: int, scale: float, window: int, keep_first: int,
                          sink: Optional[float], gate: Optional[torch.Tensor], gate_off: int, out_scale: float,
                          status: Optional[torch.Tensor] = None, items: Optional[torch.Tensor] = None,
-                         n_items: Optional[int] = None, gate_heads: bool = False) -> torch.Tensor:
+                         n_items: Optional[int] = None, gate_heads: bool = False, chunk: int = 0) -> torch.Tensor:
     """The same attention token by token in bfloat16, one block per (token, key/value head) for all the query heads
     that read it; ``items`` as for the plain kernel."""
     if not (q.dtype == torch.bfloat16 and bool(lib().st_gqa_attention_single_applies(nh, nkv, dim, vd))):
@@ -1451,7 +1547,7 @@ def gqa_attention_single(q: torch.Tensor, pool: torch.Tensor, layer: int, out: t
                                          _p(seq_of_token), _p(slots), _p(block_table), block_table.shape[1], n, nh, nkv,
                                          dim, vd, page_size, _f(scale), window, keep_first, has_sink,
                                          sink_one, gate_ptr, gate_ld, _f(out_scale), _p(status), _stream(), sinks,
-                                         int(gate_heads)), "gqa_attention_single")
+                                         int(gate_heads), chunk), "gqa_attention_single")
     return out
 
 

@@ -26,7 +26,7 @@ TIMED = ("embed", "add_positions", "add_norm", "bias_act", "scatter_i32", "gathe
          "moe_combine", "concat_rows", "scale_softcap", "gqa_prepare", "gqa_attention_plain", "gqa_attention_single",
          "gqa_attention_tiles", "delta_rule", "gated_clamped_act", "hc_spread", "hc_sum", "hc_read_norm", "hc_write", "hc_write_read_norm", "hc_step_conv",
          "norm_pair_sum", "xielu", "conv_act", "gated_norm_add", "side_input", "slice_rows", "mamba_scan", "mamba_single",
-         "moe_choose", "talk_attention_plain", "talk_attention_tiles", "talk_attention_single")
+         "moe_choose", "scaled_sum_norms", "gqa_prepare_whole_norm", "talk_attention_plain", "talk_attention_tiles", "talk_attention_single")
 
 _originals: Dict[str, object] = {}
 _events: List[Tuple[str, torch.cuda.Event, torch.cuda.Event]] = []

@@ -9,8 +9,12 @@ norm_after (the norm on the sub-layer's output only; the sub-layers read x itsel
     r = x + mult * norm1(mixer(x));  x' = r + mult * norm2(ffn(r))
 parallel  (one norm, both sub-layers read its output):
     h = norm1(x);  x' = x + (mixer(h) + ffn(h))
+parallel_scaled (a norm for each sub-layer, both of the same x, and a factor per column on each result):
+    x' = x + (a * mixer(norm1(x)) + b * ffn(norm2(x)))
 reentry   (no sub-layers; opens a pass over a stretch of layers that runs several times):
     x' = W [x ; x0] + step[turn]         x0: the embedding's rows, turn: the number of the pass
+reentry_add (no sub-layers; opens such a pass by a sum):
+    x' = x + x0
 hyper_pre_norm (n copies x_1..x_n of the residual rows instead of one; sub-layer f with coefficients a, b, M):
     u = sum_s a_s x_s;  y = f(c(norm(u)));  x_t' = sum_s M[s, t] x_s + b_t y        c: an optional short
     convolution over time, c(h) = h + conv(h); the model's residual rows are the sum of the copies
@@ -48,6 +52,25 @@ class ResidualStream:
     # (y [N, width], gate logits or None, gate bias or None, gain [width], eps): x is still to be given
     # gain * rms_unit(y * sigmoid(gate + bias)) by the next reader
     normed_pending: Optional[tuple] = None
+    # (a, a's factors, f, f's factors): x is still to be given a_scale * a + f_scale * f by the next reader.  a and f are
+    # float rows [N, width]; f may be an ops.ExpertSum or None
+    scaled_pending: Optional[tuple] = None
+    carry: Optional[torch.Tensor] = None   # float rows the same reader adds first (only beside ``scaled_pending``)
+    embedded: Optional[torch.Tensor] = None  # the embedding's rows in float (models that ask for them so)
+
+    def settle_scaled(self, positions: Optional[torch.Tensor] = None, norm1: Optional[Norm] = None,
+                      out1: Optional[torch.Tensor] = None, norm2: Optional[Norm] = None,
+                      out2: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> None:
+        """Add the two scaled results that the last block left pending (if any) to x and, in the same pass, norm the new
+        rows for their readers: out1 = norm1(x), out2 = norm2(x).  With ``rows`` only the outputs of these rows are
+        made and x, with what is pending, stays as it is."""
+        a, a_scale, f, f_scale = self.scaled_pending if self.scaled_pending is not None else (None,) * 4
+        items = f if isinstance(f, ops.ExpertSum) else None
+        ops.scaled_sum_norms(self.x, norm1.eps if norm1 is not None else 0.0, a, a_scale, None if items is not None else f,
+                             f_scale, self.carry, items, norm1.gamma if norm1 is not None else None, out1,
+                             norm2.gamma if norm2 is not None else None, out2, positions, rows)
+        if rows is None:
+            self.scaled_pending, self.carry, self.act = None, None, None
 
     def settle_normed(self, ctx: Any = None, norm: Optional[Norm] = None, out_act: Optional[torch.Tensor] = None) -> None:
         """Add the normed result that the last sub-layer left pending to x; in the same pass, with ``out_act``, what
@@ -71,6 +94,8 @@ class ResidualStream:
         stay as they are."""
         if self.normed_pending is not None:
             self.settle_normed()
+        if self.scaled_pending is not None:
+            self.settle_scaled()
         if self.lanes is not None:
             self.settle_lanes()
             ops.hc_sum(self.lanes, out=self.x)
@@ -80,6 +105,8 @@ class ResidualStream:
         """x + pending in the activation dtype (all rows, folding pending into x; or only ``rows``)."""
         if self.normed_pending is not None:
             self.settle_normed()
+        if self.scaled_pending is not None:
+            self.settle_scaled()
         if rows is None and self.pending is None and self.act is not None:
             return self.act
         n = rows.numel() if rows is not None else self.x.shape[0]
@@ -227,6 +254,91 @@ class ParallelBlock(Block):
                 ops.add_norm(stream.x, delta=a.value, resid_out=stream.x, kind="none", act_dtype=stream.act_dtype)
                 pending = f
         stream.pending, stream.act = pending, None
+
+
+@BLOCKS.register("parallel_scaled")
+class ParallelScaledBlock(Block):
+    """x <- x + (a * mixer(norm1(x)) + b * ffn(norm2(x))): both sub-layers read the same x through RMS norms of their own
+    (of one eps), and their results are multiplied by factors per column, the tensors ``scale_names`` (a, b).  The
+    feed-forward may be absent (and norm2 and b with it).  The results are left pending
+    (``ResidualStream.scaled_pending``): the next reader's kernel scales and sums them, a mixture's experts among them,
+    and makes both norms of its own rows in one pass.  Sums, factors and norm statistics are float."""
+
+    def __init__(self, mixer: Mixer, feed_forward: Optional[FeedForward], norm1: Norm, norm2: Optional[Norm], width: int,
+                 scale_names: tuple):
+        if (feed_forward is None) != (norm2 is None):
+            raise ValueError("a block has a second norm exactly when it has a feed-forward")
+        for n in (norm1, norm2):
+            if n is not None and (n.kind != "rmsnorm" or n.eps != norm1.eps):
+                raise ValueError("parallel_scaled takes RMS norms of one eps")
+        super().__init__(mixer, feed_forward, norm1, norm2)
+        self.width, self.scale_names = int(width), tuple(scale_names)[:1 if feed_forward is None else 2]
+        self.scales = [None, None]
+
+    def children(self) -> List[Part]:
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None]
+
+    def param_specs(self):
+        from ..weights.spec import GAIN, ParamSpec
+        return [ParamSpec(name, (self.width,), GAIN) for name in self.scale_names]
+
+    def bind(self, tensors) -> None:
+        for i, name in enumerate(self.scale_names):
+            self.scales[i] = tensors[name].to(torch.float32).contiguous()
+
+    def param_bytes(self) -> int:
+        return 4 * self.width * len(self.scale_names)
+
+    @staticmethod
+    def _float_rows(delta: Delta, stream: ResidualStream) -> torch.Tensor:
+        if delta.bias is None and delta.parts is None and delta.value.dtype == torch.float32:
+            return delta.value
+        y = torch.zeros(stream.x.shape, dtype=torch.float32, device=stream.x.device)
+        ops.add_norm(y, delta=delta.value, delta_bias=delta.bias, parts=delta.parts, resid_out=y, kind="none",
+                     act_dtype=stream.act_dtype)
+        return y
+
+    def forward(self, stream: ResidualStream, ctx: Any, cache: Any) -> None:
+        if stream.pending is not None or stream.normed_pending is not None:
+            stream.materialise()
+        make = lambda: torch.empty(stream.x.shape, dtype=stream.act_dtype, device=stream.x.device)
+        h1, h2 = make(), make() if self.feed_forward is not None else None
+        stream.settle_scaled(ctx.positions, self.norm1, h1, self.norm2, h2)
+        a = self._float_rows(self.mixer.forward(h1, ctx, cache), stream)
+        f = None
+        if self.feed_forward is not None:
+            unsummed = getattr(self.feed_forward, "forward_unsummed", None)
+            f = unsummed(h2, ctx) if unsummed is not None else None
+            if f is None:
+                f = self._float_rows(self.feed_forward.forward(h2, ctx), stream)
+        stream.scaled_pending = (a, self.scales[0], f, self.scales[1])
+        stream.pending, stream.act = None, None
+
+
+@BLOCKS.register("reentry_add")
+class ReentryAddBlock(Block):
+    """Opens a pass over a stretch of layers that runs several times with the same weights: x <- x + x0 with x0 the
+    embedding's rows, in float (``ResidualStream.embedded``).  Where the block before left scaled results pending, the
+    sum is left to the same reader.  It has no mixer, no cache, no norm and no tensors."""
+
+    wants_embedding = "float"
+
+    def __init__(self):
+        super().__init__(None, None, None, None)
+
+    def children(self) -> List[Part]:
+        return []
+
+    def forward(self, stream: ResidualStream, ctx: Any, cache: Any) -> None:
+        if stream.embedded is None:
+            raise RuntimeError("this block needs the embedding's rows (ResidualStream.embedded)")
+        if stream.scaled_pending is not None and stream.carry is None:
+            stream.carry = stream.embedded
+            return
+        if stream.pending is not None or stream.normed_pending is not None or stream.scaled_pending is not None:
+            stream.materialise()
+        ops.add_norm(stream.x, parts=stream.embedded.unsqueeze(0), resid_out=stream.x, kind="none", act_dtype=stream.act_dtype)
+        stream.act = None
 
 
 @BLOCKS.register("reentry")

@@ -18,10 +18,12 @@ from .base import FEED_FORWARDS, Delta, FeedForward, RowTaker, stack_rows
 
 @FEED_FORWARDS.register("dense")
 class DenseFFN(FeedForward):
-    """The matrices are the tensors ``fc1_name`` / ``fc2_name`` + ``weight_suffix``."""
+    """The matrices are the tensors ``fc1_name`` / ``fc2_name`` + ``weight_suffix``.  ``float_out``: the second product
+    leaves its float sums as they are."""
 
     def __init__(self, hidden: int, inner: int, activation: str, fc1_name: str, fc2_name: str, bias: bool = True,
-                 weight_suffix: str = ".weight"):
+                 weight_suffix: str = ".weight", float_out: bool = False):
+        self.float_out = bool(float_out)
         if activation not in ops.ACT_CODES:
             raise ValueError(f"activation '{activation}' is not supported ({', '.join(ops.ACT_CODES)})")
         self.hidden, self.inner, self.activation, self.bias = hidden, inner, activation, bias
@@ -46,6 +48,8 @@ class DenseFFN(FeedForward):
 
     def forward(self, h: torch.Tensor, ctx: Any) -> Delta:
         u = ops.linear(h, self.w1, self.b1, self.activation, bias_bf16=self.b1_bf16)
+        if self.float_out:
+            return Delta(ops.linear(u, self.w2, out_dtype=torch.float32), self.b2)
         if u.shape[0] > ops.SKINNY_MAX_ROWS and ops.linear_parts_slices(u.shape[0], self.w2) > 1:
             # fc2 for this many tokens is cut over k: its slices' sums are left for the next norm kernel
             return Delta(None, self.b2, ops.linear_parts(u, self.w2))

@@ -6,8 +6,11 @@ Per query head a (key/value head a // (heads / kv_heads)), key/query size ``dim`
     q, k      <- rotated by position on the first ``rot.dims`` dimensions (a rotary encoding: halves or pairs), or not
     q         <- q * (1 + coef * ln(floor((p + 1) / every) + 1))            (``q_temp`` = (coef, every), or None)
     s_j       = scale * q . k_j  over the keys the query at p sees: j <= p, and with a ``window``
-                p - j < window or j < keep_first
+                p - j < window or j < keep_first; with ``chunk`` only keys of the query's own run of ``chunk``
+                positions, floor(j / chunk) = floor(p / chunk)
     q, k      <- q / rms(q), k / rms(k) over ``dim``, after the rotation   (``qk_norm_eps``, or None)
+                 with ``qk_norm_names``: before the rotation, q over the root mean square of all query heads' numbers
+                 together times a weight per number, k likewise over all key heads'
     w_j       = exp(s_j) / (sum_i exp(s_i) [+ exp(sink)])                  (``sink``: a logit, or None; ``sink_name``:
                                                                             a learned logit per head)
     w_a(j)    <- sum_b T[a, b] w_b(j)                                      (``talk_name``: T [heads, heads] mixes the
@@ -17,7 +20,8 @@ Per query head a (key/value head a // (heads / kv_heads)), key/query size ``dim`
                                                                             True: a number per (head, value dimension),
                                                                             "head": one number per head)
 
-and the heads' results go through the output projection.  ``own_kv`` False: the mixer has no key and value
+and the heads' results go through the output projection.  ``values_are_keys``: there is no value projection, the
+values are the keys as projected (bias in, before norm and rotation).  ``own_kv`` False: the mixer has no key and value
 projections and reads the pages another layer step fills (the model's layer order points it at that entry).
 
 The cache holds, per key/value head and position, the key (after bias and rotation) and the value, in pages
@@ -33,14 +37,14 @@ from typing import Any, Dict, List, Optional, Tuple
 import torch
 
 from .. import ops
-from ..weights.spec import MATRIX, VECTOR, ParamSpec
+from ..weights.spec import GAIN, MATRIX, VECTOR, ParamSpec
 from .attention import PagedAttentionPlan
 from .base import MIXERS, Delta, Mixer, PagedKVSpec, RowTaker, StepPlan, stack_rows
 
 
 @MIXERS.register("grouped_attention")
 class GroupedAttention(RowTaker, Mixer):
-    """names: tensor names of the projections {"q","k","v","o"} and, with ``gate``, "g" ([out, in] matrices);
+    """names: tensor names of the projections {"q","k","v","o"} (no "v" with ``values_are_keys``) and, with ``gate``, "g" ([out, in] matrices);
     a projection's bias is its name + ``bias_suffix``.  ``qkv_bias`` / ``o_bias``: which projections have one."""
 
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float,
@@ -48,7 +52,15 @@ class GroupedAttention(RowTaker, Mixer):
                  window: Optional[int] = None, keep_first: int = 0, sink: Optional[float] = None,
                  qk_position: Any = None, q_temp: Optional[Tuple[float, int]] = None, gate: Any = False,
                  out_scale: float = 1.0, own_kv: bool = True, sink_name: Optional[str] = None,
-                 talk_name: Optional[str] = None, qk_norm_eps: Optional[float] = None, float_out: bool = False):
+                 talk_name: Optional[str] = None, qk_norm_eps: Optional[float] = None, float_out: bool = False,
+                 chunk: Optional[int] = None, values_are_keys: bool = False,
+                 qk_norm_names: Optional[Tuple[str, str]] = None):
+        if chunk is not None and (chunk <= 0 or talk_name):
+            raise ValueError("a chunk holds at least one key, and heads are not mixed under it")
+        if values_are_keys and (vdim != dim or not own_kv):
+            raise ValueError("values that are the keys have their size, and the mixer its own keys")
+        if qk_norm_names and (not qk_norm_eps or not own_kv):
+            raise ValueError("norms over whole projections need 'qk_norm_eps' and the mixer's own keys")
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads cannot share {num_kv_heads} key/value heads")
         if window is not None and window <= 0:
@@ -75,9 +87,12 @@ class GroupedAttention(RowTaker, Mixer):
         self.float_out = bool(float_out)
         self.qw = num_heads * dim
         self.kw = num_kv_heads * dim if own_kv else 0
-        self.vw = num_kv_heads * vdim if own_kv else 0
+        self.vw = num_kv_heads * vdim if own_kv and not values_are_keys else 0      # columns of a value projection
+        self.v_off = self.qw if values_are_keys else self.qw + self.kw
+        self.chunk, self.qk_norm_names = (int(chunk) if chunk else None), (tuple(qk_norm_names) if qk_norm_names else None)
         self.gw = (num_heads if self.gate_heads else num_heads * vdim) if gate else 0
         self.w_in = self.b_in = self.w_o = self.b_o = self.sinks = self.talk = None
+        self.q_norm = self.k_norm = None
         self._plan: Optional[PagedAttentionPlan] = None
         self.extra_off = self.extra_n = 0
 
@@ -85,7 +100,7 @@ class GroupedAttention(RowTaker, Mixer):
     def _projections(self):
         out = [("q", self.qw)]
         if self.own_kv:
-            out += [("k", self.kw), ("v", self.vw)]
+            out += [("k", self.kw)] + ([("v", self.vw)] if self.vw else [])
         if self.gate:
             out.append(("g", self.gw))
         return out
@@ -103,6 +118,8 @@ class GroupedAttention(RowTaker, Mixer):
             specs.append(ParamSpec(self.sink_name, (self.nh,), VECTOR))
         if self.talk_name:
             specs.append(ParamSpec(self.talk_name, (self.nh, self.nh), VECTOR))
+        if self.qk_norm_names:
+            specs += [ParamSpec(name, (rows,), GAIN) for name, rows in zip(self.qk_norm_names, (self.qw, self.kw))]
         return specs
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -127,13 +144,15 @@ class GroupedAttention(RowTaker, Mixer):
             self.sinks = tensors[self.sink_name].to(torch.float32).contiguous()
         if self.talk_name:
             self.talk = tensors[self.talk_name].to(torch.float32).contiguous()
+        if self.qk_norm_names:
+            self.q_norm, self.k_norm = (tensors[name].to(torch.float32).contiguous() for name in self.qk_norm_names)
 
     def param_bytes(self) -> int:
         return (self.w_in.numel() + self.w_o.numel()) * self.w_in.element_size()
 
     # ------------------------------------------------------------ cache, plan
     def cache_spec(self) -> PagedKVSpec:
-        return PagedKVSpec(self.nkv, self.dim, self.window, value_dim=self.vdim, keep_first=self.keep_first)
+        return PagedKVSpec(self.nkv, self.dim, self.window, value_dim=self.vdim, block=self.chunk, keep_first=self.keep_first)
 
     def step_plan(self) -> StepPlan:
         # the paged attention's sorting of a step's tokens: portions in tiles, short ones and single tokens as items
@@ -150,11 +169,15 @@ class GroupedAttention(RowTaker, Mixer):
         rot_dims = rot.dims if rot is not None else 0
         temp = self.q_temp or (0.0, 1)
         ps = cache.page_size
-        ops.gqa_prepare(proj, 0, self.qw, self.qw + self.kw, self.b_in, rot.inv_freq(h.device) if rot_dims else None,
-                        rot_dims, temp[0], temp[1], q, cache.pool, cache.layer, ctx.positions, ctx.seq_of_token,
-                        ctx.slots, cache.block_table, self.nh, self.nkv, self.dim, self.vdim, ps, ctx.status,
-                        write_kv=self.own_kv and cache.writable, norm_eps=self.qk_norm_eps,
-                        neighbours=rot is not None and rot.neighbours, rot_amp=rot.amplitude if rot is not None else 1.0)
+        args = (proj, 0, self.qw, self.v_off, self.b_in, rot.inv_freq(h.device) if rot_dims else None, rot_dims, temp[0],
+                temp[1], q, cache.pool, cache.layer, ctx.positions, ctx.seq_of_token, ctx.slots, cache.block_table, self.nh,
+                self.nkv, self.dim, self.vdim, ps, ctx.status)
+        turn = dict(write_kv=self.own_kv and cache.writable, neighbours=rot is not None and rot.neighbours,
+                    rot_amp=rot.amplitude if rot is not None else 1.0)
+        if self.qk_norm_names:
+            ops.gqa_prepare_whole_norm(*args, self.q_norm, self.k_norm, self.qk_norm_eps, **turn)
+        else:
+            ops.gqa_prepare(*args, norm_eps=self.qk_norm_eps, **turn)
         extra = proj[:, self.extra_off:self.extra_off + self.extra_n] if self.extra_n else None
         o = torch.empty((n, self.nh * self.vdim), dtype=h.dtype, device=h.device)
         gate, gate_off = (proj, self.qw + self.kw + self.vw) if self.gate else (None, 0)
@@ -193,14 +216,15 @@ class GroupedAttention(RowTaker, Mixer):
             if plan.n_tiles:
                 ops.gqa_attention_tiles(q, cache.pool, cache.layer, o, plan.tiles, plan.n_tiles, self._plan.tile_rows,
                                         ctx.q_start, ctx.start_pos, ctx.slots, cache.block_table, *consts,
-                                        status=ctx.status, gate_heads=self.gate_heads)
+                                        status=ctx.status, gate_heads=self.gate_heads, chunk=self.chunk or 0)
             if plan.n_items:
                 ops.gqa_attention_single(q, cache.pool, cache.layer, o, ctx.positions, ctx.seq_of_token, ctx.slots,
                                          cache.block_table, *consts, status=ctx.status, items=plan.items,
-                                         n_items=plan.n_items, gate_heads=self.gate_heads)
+                                         n_items=plan.n_items, gate_heads=self.gate_heads, chunk=self.chunk or 0)
         else:
             ops.gqa_attention_plain(q, cache.pool, cache.layer, o, ctx.positions, ctx.seq_of_token, ctx.slots,
-                                    cache.block_table, *consts, status=ctx.status, gate_heads=self.gate_heads)
+                                    cache.block_table, *consts, status=ctx.status, gate_heads=self.gate_heads,
+                                    chunk=self.chunk or 0)
         return Delta(ops.linear(o, self.w_o, out_dtype=torch.float32 if self.float_out else None), self.b_o, extra=extra)
 
     def _sink_vector(self, device) -> Optional[torch.Tensor]:

@@ -77,12 +77,16 @@ class RotaryPairs(PositionEncoding):
         turns(t) = dims * ln(original / (2 pi t)) / (2 ln base), the index at which a pair turns t times within
         ``original`` positions, pairs before floor(turns(fast)) keep their frequency, those after ceil(turns(slow)) turn
         ``factor`` times slower, a linear ramp lies between, and sine and cosine are multiplied by
-        0.1 ln(factor) + 1 (``amplitude``)."""
+        0.1 ln(factor) + 1 (``amplitude``).  Or {"factor", "original", "low", "high"}, a stretch by wavelength: with
+        the wavelength l = 2 pi / f of a pair, pairs with l < original / high keep their frequency, those with
+        l > original / low turn ``factor`` times slower, in between the two are mixed with the share
+        (original / l - low) / (high - low) of the kept frequency; the amplitude stays 1."""
         if dims < 0 or dims % 2:
             raise ValueError(f"rotary dimensions must be even and not negative, got {dims}")
         self.dims, self.base = int(dims), float(base)
         self.scaling = dict(scaling) if scaling else None
-        self.amplitude = 0.1 * math.log(self.scaling["factor"]) + 1.0 if self.scaling else 1.0
+        self._by_wavelength = bool(self.scaling) and "low" in self.scaling
+        self.amplitude = 0.1 * math.log(self.scaling["factor"]) + 1.0 if self.scaling and not self._by_wavelength else 1.0
         self._tables: Dict[torch.device, torch.Tensor] = {}
 
     def frequencies(self) -> List[float]:
@@ -91,6 +95,8 @@ class RotaryPairs(PositionEncoding):
         if not self.scaling:
             return f
         s = self.scaling
+        if self._by_wavelength:
+            return [self._stretched(v) for v in f]
         turns = lambda t: self.dims * math.log(s["original"] / (2.0 * math.pi * t)) / (2.0 * math.log(self.base))
         lo, hi = max(math.floor(turns(s["fast"])), 0), min(math.ceil(turns(s["slow"])), self.dims - 1)
         out = []
@@ -98,6 +104,15 @@ class RotaryPairs(PositionEncoding):
             ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
             out.append(v / s["factor"] * ramp + v * (1.0 - ramp))
         return out
+
+    def _stretched(self, f: float) -> float:
+        s, wavelength = self.scaling, 2.0 * math.pi / f
+        if wavelength < s["original"] / s["high"]:
+            return f
+        if wavelength > s["original"] / s["low"]:
+            return f / s["factor"]
+        kept = (s["original"] / wavelength - s["low"]) / (s["high"] - s["low"])
+        return (1.0 - kept) * f / s["factor"] + kept * f
 
     def inv_freq(self, device) -> torch.Tensor:
         device = torch.device(device)
