@@ -13,7 +13,7 @@ single-GPU and exits with 2.
 ``--only decode|prefill`` run one small measurement (for profiling); ``--only mixed`` runs a continuous
 batch of requests of random lengths (prompt portions of 512 tokens beside decoded tokens) through
 ``LLMEngine.generate`` and reports tokens per second, steps and preemptions.  ``--only designs`` measures a
-Fanidra, a Pikadra, a Norelix, a Nafelix and a Nigilorn model beside an OPT model of equal width, depth and parameter count (prefill, decode,
+Fanidra, a Pikadra, a Norelix, a Nafelix, a Nigilorn and a Dimalix model beside an OPT model of equal width, depth and parameter count (prefill, decode,
 and the device time of every operation of one step of each kind; ``--model-name w2048|w4096`` picks one size,
 ``--layers`` the depth, ``--designs`` which of the six).
 """
@@ -118,6 +118,11 @@ def prefill_flops(cfg, n_layers, n):
 # a sixteenth of the width, four taps) with mixtures of eight two-matrix experts in four groups (three kept), two per
 # token, and a shared expert, each one and a half times as wide as Pikadra's three-matrix ones (the same parameter count);
 # one layer of grouped attention with the Norelix pair's sizes and a window as long as the context.
+# The Dimalix model of a size: the Nigilorn model's latent attention in three of four layers, the last one grouped attention
+# whose values are its keys (the Norelix pair's heads, keys as wide as its values, chunks of 512); the first layer has a
+# dense two-matrix feed-forward one and a half times as wide as Pikadra's three-matrix one, the others twelve experts of
+# Pikadra's size and four identity outputs in four groups (two kept), four choices per token (the same parameter count
+# as Pikadra's experts and shared expert).
 DESIGN_SIZES = {
     "w2048": dict(width=2048, opt_heads=32, opt_ffn=8192, heads=16, kv_heads=4, dim=64, vdim=128, ff=5504,
                   rec_heads=16, rec_dim=128, rec_vdim=128, block=512,
@@ -132,13 +137,13 @@ DESIGN_SIZES = {
 
 def compare_designs(args, peaks):
     """Prefill (2048 tokens) and decode (batch 8 behind 512-token prompts) of a Fanidra, a Pikadra, a Norelix, a Nafelix, a
-    Nigilorn and an OPT model of equal size, random weights, device-timed; and the device time of every operation of one prefill step and one
-    decode step launched kernel by kernel.  One JSON line per (size, design)."""
+    Nigilorn, a Dimalix and an OPT model of equal size, random weights, device-timed; and the device time of every operation of
+    one prefill step and one decode step launched kernel by kernel.  One JSON line per (size, design)."""
     import gc
     import numpy as np
     import torch
     from swifttransformer_b200 import ops
-    from swifttransformer_b200.config import (FanidraConfig, NafelixConfig, NigilornConfig, NorelixConfig, OptConfig,
+    from swifttransformer_b200.config import (DimalixConfig, FanidraConfig, NafelixConfig, NigilornConfig, NorelixConfig, OptConfig,
                                               PikadraConfig)
     from swifttransformer_b200.engine.engine import LLMEngine
     from swifttransformer_b200.engine.step import StepEntry
@@ -209,7 +214,18 @@ def compare_designs(args, peaks):
         nig = NigilornConfig.from_dict(dict(architecture="Nigilorn", vocab=vocab, width=z["width"], norm={"eps": 1e-6},
                                             token_side={"dim": 64}, layers=[(ng_lat, ng_ssm, ng_ssm, ng_att)[i % 4]
                                                                             for i in range(n_layers)]))
-        all_designs = {"fanidra": fan, "pikadra": pik, "norelix": nor, "nafelix": naf, "nigilorn": nig, "opt": opt}
+        by_wave = {"factor": 8.0, "original": 2048, "low": 1.0, "high": 4.0}
+        dm_moe = {"kind": "moe", "expert": {"ff": k["expert_ff"]},
+                  "router": {"experts": 12, "identity": 4, "top": 4, "groups": {"count": 4, "keep": 2}}}
+        dm_mix = dict(ng_lat["mixer"], rot={"dims": k["rot"], "base": 10000.0})
+        dm_att = {"type": "attention", "mlp": dm_moe,
+                  "mixer": dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["vdim"], vdim=z["vdim"], scale=z["vdim"] ** -0.5,
+                                mask={"size": z["block"]}, rot={"dims": z["vdim"], "base": 10000.0, "scaling": by_wave})}
+        dm_lat = lambda mlp: {"type": "latent_attention", "mixer": dm_mix, "mlp": mlp}
+        dm_layers = (dm_lat({"kind": "dense", "ff": k["ff"] * 3 // 2}), dm_lat(dm_moe), dm_lat(dm_moe), dm_att)
+        dim = DimalixConfig.from_dict(dict(architecture="Dimalix", vocab=vocab, width=z["width"], norm={"eps": 1e-6},
+                                           embedding={"scale": 8.0}, layers=[dm_layers[i % 4] for i in range(n_layers)]))
+        all_designs = {"dimalix": dim, "fanidra": fan, "pikadra": pik, "norelix": nor, "nafelix": naf, "nigilorn": nig, "opt": opt}
         return {d: c for d, c in all_designs.items() if not args.designs or d in args.designs.split(",")}
 
     def engine(model, graphs=True):
@@ -312,7 +328,7 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=512)
     ap.add_argument("--layers", type=int, default=0, help="run fewer layers than the model has (0: all)")
     ap.add_argument("--designs", default="", help="with --only designs: which designs to measure, with commas between "
-                    "them (fanidra, pikadra, norelix, nafelix, nigilorn, opt; default: all)")
+                    "them (fanidra, pikadra, norelix, nafelix, nigilorn, dimalix, opt; default: all)")
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 and prefill measurements")
     ap.add_argument("--no-big", action="store_true", help="skip the OPT-6.7B and OPT-30B points (13 and 60 GB of random weights)")
     ap.add_argument("--launch-floor", action="store_true",

@@ -105,7 +105,7 @@ class DimalixConfig(ModelConfig):
             loop = tuple(_need(raw["loop"], key, "loop.", int) for key in ("start", "stop", "times"))
         cfg = cls(vocab=_need(raw, "vocab", "", int), width=_need(raw, "width", "", int),
                   layers=tuple(copy.deepcopy(layers)), norm_eps=float(_need(raw.get("norm"), "eps", "norm.")),
-                  embedding_scale=float(_need(raw["embedding"], "scale", "embedding.")) if raw.get("embedding") else 1.0,
+                  embedding_scale=float(_need(raw["embedding"], "scale", "embedding.")) if raw.get("embedding") is not None else 1.0,
                   loop=loop)
         cfg.validate()
         return cfg

@@ -136,7 +136,7 @@ gqa_prepare_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
 // squares in one walk over the row, then queries, keys and values.  VEC: neighbours are paired, and rows, heads and
 // weights allow pieces of four; else one element at a time in either layout.
 template <typename T, bool VEC>
-__global__ void __launch_bounds__(GP_THREADS)
+__global__ void __launch_bounds__(2 * GP_THREADS)
 gqa_prepare_whole_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, int v_off,
                               const float* __restrict__ bias, Rotation rot, float temp_coef, int temp_every,
                               const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
@@ -159,7 +159,7 @@ gqa_prepare_whole_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int
         if (page < 0 && status && threadIdx.x == 0) *status = 1;
     }
     const int pip = pos % cache.page_size;
-    for (int i = threadIdx.x; i < rot.dims / 2; i += GP_THREADS) {
+    for (int i = threadIdx.x; i < rot.dims / 2; i += blockDim.x) {
         float sn, cs;
         sincosf((float)pos * rot.freq[i], &sn, &cs);
         turn[i] = make_float2(cs * rot.amp, sn * rot.amp);
@@ -172,7 +172,7 @@ gqa_prepare_whole_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int
     };
     constexpr int STEP = VEC ? 4 : 1;
     float sq = 0.f, sk = 0.f;
-    for (int c = threadIdx.x * STEP; c < qw + kw; c += GP_THREADS * STEP) {
+    for (int c = threadIdx.x * STEP; c < qw + kw; c += blockDim.x * STEP) {
         const bool is_q = c < qw;
         const int col = is_q ? q_off + c : k_off + c - qw;
         float d;
@@ -188,7 +188,7 @@ gqa_prepare_whole_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int
     const float rq = rsqrtf(block_sum(sq, scratch) / (float)qw + eps);       // (its barriers also publish `turn`)
     const float rk = kw > 0 ? rsqrtf(block_sum(sk, scratch) / (float)kw + eps) : 0.f;
     const float temp = temp_coef != 0.f ? 1.f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.f) : 1.f;
-    for (int c = threadIdx.x * STEP; c < qw + kw; c += GP_THREADS * STEP) {
+    for (int c = threadIdx.x * STEP; c < qw + kw; c += blockDim.x * STEP) {
         const bool is_q = c < qw;
         if (!is_q && page < 0) continue;
         const int cc = is_q ? c : c - qw, head = cc / dim, e = cc % dim;
@@ -223,7 +223,7 @@ gqa_prepare_whole_norm_kernel(const T* __restrict__ proj, int ld, int q_off, int
         }
     }
     if (page < 0) return;
-    for (int c = threadIdx.x * STEP; c < vw; c += GP_THREADS * STEP) {
+    for (int c = threadIdx.x * STEP; c < vw; c += blockDim.x * STEP) {
         T* dst = cache_values(pool, cache, page, c / vd, pip) + c % vd;
         if (VEC) store4(dst, at4(v_off + c));
         else *dst = from_f32<T>(at(v_off + c));
@@ -249,9 +249,11 @@ ST_EXPORT int st_gqa_prepare_whole_norm(const void* proj, int ld, int q_off, int
     const bool vec = (neighbours || rot_dims == 0) && dim % 4 == 0 && vd % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 &&
                      k_off % 4 == 0 && v_off % 4 == 0 && page_stride % 4 == 0 && entry_offset % 4 == 0 && aligned16(proj) &&
                      aligned16(bias) && aligned16(q_w) && aligned16(k_w) && aligned16(q_out) && aligned16(pool);
+    // steps of few tokens: more threads per token, so that its row is asked for at once
+    const int threads = n_tokens < st_sm_count() ? 2 * GP_THREADS : GP_THREADS;
     cudaStream_t s = (cudaStream_t)stream;
 #define GW_LAUNCH(T, VEC)                                                                                                 \
-    return st_launch_pdl("gqa_prepare", gqa_prepare_whole_norm_kernel<T, VEC>, dim3(n_tokens), dim3(GP_THREADS), smem, s, \
+    return st_launch_pdl("gqa_prepare", gqa_prepare_whole_norm_kernel<T, VEC>, dim3(n_tokens), dim3(threads), smem, s, \
                          (const T*)proj, ld, q_off, k_off, v_off, bias, rot, temp_coef, temp_every, q_w, k_w, eps,        \
                          (T*)q_out, (T*)pool, c, positions, seq_of_token, slots, block_table, nh, write_kv, status)
     if (dtype == 0) {

@@ -21,7 +21,7 @@
 //              With identity experts: + h[t] times the sum of the weights whose expert is n_real or above.
 #include "moe.cuh"
 
-#define ROUTE_THREADS 256
+#define ROUTE_MAX_THREADS 1024     // a warp per router output up to this many
 #define ROUTE_MAX_EXPERTS 1024
 
 struct RouteRule {
@@ -105,7 +105,7 @@ __device__ __forceinline__ void route_choose(float* z, int n_experts, int top, c
 }
 
 template <typename T>
-__global__ void __launch_bounds__(ROUTE_THREADS)
+__global__ void __launch_bounds__(ROUTE_MAX_THREADS)
 moe_route_kernel(const T* __restrict__ h, int width, const float* __restrict__ w_r, int n_experts, int top,
                  RouteRule rule, const float* __restrict__ w_g, const int* __restrict__ positions,
                  int* __restrict__ experts, float* __restrict__ weights, float* __restrict__ gate, int vec) {
@@ -113,9 +113,9 @@ moe_route_kernel(const T* __restrict__ h, int width, const float* __restrict__ w
     ST_PDL_WAIT();
     ST_PDL_TRIGGER();
     const int t = blockIdx.x;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = ROUTE_THREADS / 32;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x / 32;
     if (positions && positions[t] < 0) {
-        for (int k = threadIdx.x; k < top; k += ROUTE_THREADS) { experts[(size_t)t * top + k] = -1; weights[(size_t)t * top + k] = 0.f; }
+        for (int k = threadIdx.x; k < top; k += blockDim.x) { experts[(size_t)t * top + k] = -1; weights[(size_t)t * top + k] = 0.f; }
         if (gate && threadIdx.x == 0) gate[t] = 0.f;
         return;
     }
@@ -126,6 +126,7 @@ moe_route_kernel(const T* __restrict__ h, int width, const float* __restrict__ w
         float d = 0.f;
         if (vec) {
             // four at a time; a lane's partial sums run in the same order whatever the batch
+#pragma unroll 8
             for (int i = lane * 4; i < width; i += 128) {
                 const float4 a = load4_cg(row + i), c = *reinterpret_cast<const float4*>(wr + i);
                 d = fmaf(a.x, c.x, fmaf(a.y, c.y, fmaf(a.z, c.z, fmaf(a.w, c.w, d))));
@@ -190,11 +191,13 @@ ST_EXPORT int st_moe_route(const void* h, int n_tokens, int width, const float* 
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)(route_floats(n_experts, rule) + 1) * sizeof(float);
     const int vec = width % 4 == 0 && aligned16(h) && aligned16(w_r) && (!w_g || aligned16(w_g));
+    const int outputs = n_experts + (w_g ? 1 : 0);
+    const int threads = outputs * 32 > ROUTE_MAX_THREADS ? ROUTE_MAX_THREADS : outputs * 32;
     if (dtype == 0)
-        return st_launch_pdl("moe_route", moe_route_kernel<float>, dim3(n_tokens), dim3(ROUTE_THREADS), smem, s, (const float*)h,
+        return st_launch_pdl("moe_route", moe_route_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, (const float*)h,
                              width, w_r, n_experts, top, rule, w_g, positions, experts, weights, gate, vec);
     if (dtype == 1)
-        return st_launch_pdl("moe_route", moe_route_kernel<bf16>, dim3(n_tokens), dim3(ROUTE_THREADS), smem, s, (const bf16*)h,
+        return st_launch_pdl("moe_route", moe_route_kernel<bf16>, dim3(n_tokens), dim3(threads), smem, s, (const bf16*)h,
                              width, w_r, n_experts, top, rule, w_g, positions, experts, weights, gate, vec);
     return ST_ERR_BAD_DTYPE;
 }
