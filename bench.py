@@ -15,7 +15,7 @@ batch of requests of random lengths (prompt portions of 512 tokens beside decode
 ``LLMEngine.generate`` and reports tokens per second, steps and preemptions.  ``--only designs`` measures a
 Fanidra, a Pikadra, a Norelix, a Nafelix, a Nigilorn and a Dimalix model beside an OPT model of equal width, depth and parameter count (prefill, decode,
 and the device time of every operation of one step of each kind; ``--model-name w2048|w4096`` picks one size,
-``--layers`` the depth, ``--designs`` which of the six).
+``--layers`` the depth, ``--designs`` which of the seven).
 """
 import argparse
 import json

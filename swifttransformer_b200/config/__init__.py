@@ -9,4 +9,5 @@ from .opt import OptConfig, opt_preset
 from .pikadra import PikadraConfig
 
 __all__ = ["ConfigError", "DimalixConfig", "FanidraConfig", "ModelConfig", "NafelixConfig", "NigilornConfig", "NorelixConfig",
-           "OptConfig", "PikadraConfig", "config_class", "config_from_dict", "known_architectures", "load_config", "opt_preset", "register_config", "save_config"]
+           "OptConfig", "PikadraConfig", "config_class", "config_from_dict", "known_architectures", "load_config",
+           "opt_preset", "register_config", "save_config"]

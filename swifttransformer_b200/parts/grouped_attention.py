@@ -44,8 +44,8 @@ from .base import MIXERS, Delta, Mixer, PagedKVSpec, RowTaker, StepPlan, stack_r
 
 @MIXERS.register("grouped_attention")
 class GroupedAttention(RowTaker, Mixer):
-    """names: tensor names of the projections {"q","k","v","o"} (no "v" with ``values_are_keys``) and, with ``gate``, "g" ([out, in] matrices);
-    a projection's bias is its name + ``bias_suffix``.  ``qkv_bias`` / ``o_bias``: which projections have one."""
+    """names: tensor names of the projections {"q","k","v","o"} (no "v" with ``values_are_keys``) and, with ``gate``, "g"
+    ([out, in] matrices); a projection's bias is its name + ``bias_suffix``.  ``qkv_bias`` / ``o_bias``: which projections have one."""
 
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float,
                  names: Dict[str, str], qkv_bias: bool = True, o_bias: bool = False, bias_suffix: str = ".b",
